@@ -4,7 +4,8 @@ Run entries of a model (see ``parts.spec.RunEntry``) that keep the same kind
 of cache form a *group*.  A paged group (``PagedKV``) has a page pool of its
 own; a request has one block table per paged group, and one page id stands
 for that page in every entry of the group.  A group with a window gives
-pages back as soon as every later query is past them; a group without keeps
+pages back as soon as every later query is past them, except those that hold
+the first tokens it keeps in sight (``keep_first``); a group without keeps
 them until the request ends.  A fixed-state group (``FixedState``) keeps its
 state in the request's *slot*; slots exist for every request, whether or not
 the architecture has such state.
@@ -42,13 +43,17 @@ class CacheGroup:
     def paged(self) -> bool:
         return isinstance(self.need, PagedKV)
 
+    def kept_blocks(self, page_size: int) -> int:
+        """Blocks at a request's start that no window ever passes."""
+        return -(-self.need.keep_first // page_size) if self.paged else 0
+
 
 @dataclass
 class _Request:
     slot: int
     length: int = 0                    # committed tokens
     reserved: int = 0                  # tokens pages are reserved for (>= length)
-    first_block: dict = field(default_factory=dict)   # group -> first block still held
+    first_block: dict = field(default_factory=dict)   # group -> first block still held (apart from the kept first ones)
     n_blocks: dict = field(default_factory=dict)      # group -> blocks ever appended
 
 
@@ -119,7 +124,7 @@ class CacheManager:
             if not group.paged:
                 continue
             row = group.table[slot]
-            held = [int(p) for p in row[request.first_block[group.index]:request.n_blocks[group.index]] if p != NO_PAGE]
+            held = [int(p) for p in row[:request.n_blocks[group.index]] if p != NO_PAGE]
             group.pool.free(held, slot)
             self._freed(group, held)
             row[:] = NO_PAGE
@@ -224,7 +229,7 @@ class CacheManager:
             if group.need.block is not None:
                 first_needed = max(first_needed, request.length // group.need.block * group.need.block)
             keep_from = min(first_needed // self.page_size, request.n_blocks[group.index])
-            first = request.first_block[group.index]
+            first = max(request.first_block[group.index], group.kept_blocks(self.page_size))
             if keep_from > first:
                 row = group.table[slot]
                 passed = [int(p) for p in row[first:keep_from]]
@@ -239,7 +244,11 @@ class CacheManager:
 
     def pages_held(self, slot: int) -> list:
         request = self._take(slot)
-        return [request.n_blocks[g.index] - request.first_block[g.index] if g.paged else 0 for g in self.groups]
+        held = []
+        for g in self.groups:
+            passed = max(0, request.first_block[g.index] - g.kept_blocks(self.page_size)) if g.paged else 0
+            held.append(request.n_blocks[g.index] - passed if g.paged else 0)
+        return held
 
     def pages_free(self) -> list:
         return [g.pool.available if g.paged else 0 for g in self.groups]

@@ -223,15 +223,20 @@ __device__ __forceinline__ void cp_async_16(void* smem, const void* global) {
 //   acc  [tokens, heads, max_chunks, head_size]   un-normalised weighted values
 //   ml   [tokens, heads, max_chunks, 2]           running maximum, running sum
 // and one int32 counter per (token, head), zero between launches.
-template <int D>       // head size: 16, 32, 64, 128 or 256
+// The keys a token sees are numbered without gaps: the kept first ones (those below `keep` that the window has
+// passed), then the window's; chunks are ranges of these numbers, so a chunk is full whatever lies between.
+// FULL: keys and values have D entries; else key rows have `dim` and value rows `vdim` entries (multiples of 8 up
+// to D; scratch keeps its stride D), and a lane past a row's end copies nothing and holds zeros.
+template <int D, bool FULL>       // head size: 16, 32, 64, 128 or 256
 __global__ void __launch_bounds__(128)
 split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restrict__ q, long ld_q,
                        const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                        const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
-                       const int* __restrict__ token_item, int n_heads, int n_kv_heads, int page_size, float scale,
-                       float cap, int window, int block, const float* __restrict__ gate, long ld_gate,
+                       const int* __restrict__ token_item, int n_heads, int n_kv_heads, int dim, int vdim, int page_size,
+                       float scale, float cap, int window, int block, int keep, const float* __restrict__ gate, long ld_gate,
                        const float* __restrict__ sink, int chunk, int max_chunks, float* __restrict__ part_acc,
                        float* __restrict__ part_ml, int* __restrict__ counters) {
+    if (FULL) dim = vdim = D;
     constexpr int LPK = D / 8;             // lanes per key: each lane owns 8 of the head's dimensions
     constexpr int KPW = 32 / LPK;          // keys per warp per step
     dependents_may_start();
@@ -243,15 +248,20 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
     // the first key seen: the window's, and with a mask of blocks of positions the first of the query's block
     int lo = (window > 0 && p - window + 1 > 0) ? p - window + 1 : 0;
     if (block > 0) lo = max(lo, p - p % block);
-    const int c_first = lo / chunk, c_last = p / chunk;
-    if (c < c_first || c > c_last) return;
-    const int begin = max(lo, c * chunk), end = min(p, c * chunk + chunk - 1);     // inclusive
+    const int n_kept = min(keep, lo), gap = lo - n_kept;        // key number i is position i (i < n_kept) or i + gap
+    const int n_seen = n_kept + p - lo + 1;
+    const int c_last = (n_seen - 1) / chunk;
+    if (c > c_last) return;
+    const int begin = c * chunk, end = min(n_seen, begin + chunk) - 1;             // key numbers, inclusive
     const int* bt = block_table + (long)token_item[t] * max_blocks;
     const int hk = h / (n_heads / n_kv_heads);
-    const long kv_width = (long)n_kv_heads * D;
+    const long k_width = (long)n_kv_heads * dim, v_width = (long)n_kv_heads * vdim;
+    const bool has_key = FULL || sub * 8 < dim, has_value = FULL || sub * 8 < vdim;
 
     float qf[8], acc[8];
-    unpack8(*reinterpret_cast<const uint4*>(q + (long)t * ld_q + (long)h * D + sub * 8), qf);
+    uint4 q8 = make_uint4(0u, 0u, 0u, 0u);
+    if (has_key) q8 = *reinterpret_cast<const uint4*>(q + (long)t * ld_q + (long)h * dim + sub * 8);
+    unpack8(q8, qf);
     // scores are kept in units of log2(e): exp(x) = 2^(x log2 e) costs one instruction then
     const float scale_log2 = scale * 1.4426950408889634f;
     // a cap on the scores, cap * tanh(score / cap), in the same units (cap <= 0: none)
@@ -273,18 +283,19 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
     const int trips = (end - (begin + warp * KPW)) / (8 * KPW) + 1;      // <= 0: nothing for this warp
     // pages of a power of two are the rule: shift and mask instead of a division per key
     const int page_shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;
-    const long head_offset = (long)hk * D + sub * 8;
+    const long k_offset = (long)hk * dim + sub * 8, v_offset = (long)hk * vdim + sub * 8;
     auto issue = [&](int trip) {
         if (trip < trips) {
 #pragma unroll
             for (int u = 0; u < 2; u++) {
-                const int j = first_key + trip * 8 * KPW + u * 4 * KPW;
-                if (j <= end) {
+                const int number = first_key + trip * 8 * KPW + u * 4 * KPW;
+                if (number <= end) {
+                    const int j = number < n_kept ? number : number + gap;
                     const int block = page_shift >= 0 ? j >> page_shift : j / page_size;
                     const int within = page_shift >= 0 ? j & (page_size - 1) : j % page_size;
-                    const long base = ((long)bt[block] * page_size + within) * kv_width + head_offset;
-                    cp_async_16(&ring[trip % RING][u][0][threadIdx.x], k_pages + base);
-                    cp_async_16(&ring[trip % RING][u][1][threadIdx.x], v_pages + base);
+                    const long slot = (long)bt[block] * page_size + within;
+                    if (has_key) cp_async_16(&ring[trip % RING][u][0][threadIdx.x], k_pages + slot * k_width + k_offset);
+                    if (has_value) cp_async_16(&ring[trip % RING][u][1][threadIdx.x], v_pages + slot * v_width + v_offset);
                 }
             }
         }
@@ -300,8 +311,8 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
         for (int u = 0; u < 2; u++) {
             const bool valid = first_key + trip * 8 * KPW + u * 4 * KPW <= end;
             float kf[8];
-            unpack8(ring[trip % RING][u][0][threadIdx.x], kf);
-            unpack8(ring[trip % RING][u][1][threadIdx.x], vf[u]);
+            unpack8(has_key ? ring[trip % RING][u][0][threadIdx.x] : make_uint4(0u, 0u, 0u, 0u), kf);
+            unpack8(has_value ? ring[trip % RING][u][1][threadIdx.x] : make_uint4(0u, 0u, 0u, 0u), vf[u]);
             float dot = 0.0f;
 #pragma unroll
             for (int i = 0; i < 8; i++) dot = fmaf(qf[i], kf[i], dot);
@@ -340,7 +351,7 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
     for (int w = 0; w < 4; w++)
         for (int g = 0; g < KPW; g++) big = fmaxf(big, sm_m[w][g]);
     const long cell = (((long)t * n_heads + h) * max_chunks + c);
-    for (int d = threadIdx.x; d < D; d += 128) {
+    for (int d = threadIdx.x; d < vdim; d += 128) {
         float o = 0.0f;
         for (int w = 0; w < 4; w++)
             for (int g = 0; g < KPW; g++) {
@@ -366,7 +377,7 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
     __syncthreads();
     if (threadIdx.x == 0) {
         int ticket = atomicAdd(&counters[t * n_heads + h], 1);
-        is_last = (ticket == c_last - c_first);
+        is_last = (ticket == c_last);
         if (is_last) counters[t * n_heads + h] = 0;       // ready for the next launch
     }
     __syncthreads();
@@ -374,20 +385,20 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
     __threadfence();
     const long first = ((long)t * n_heads + h) * max_chunks;
     float top = -INFINITY;
-    for (int cc = c_first; cc <= c_last; cc++) top = fmaxf(top, __ldcg(part_ml + (first + cc) * 2));
+    for (int cc = 0; cc <= c_last; cc++) top = fmaxf(top, __ldcg(part_ml + (first + cc) * 2));
     // a sink: one more term exp(sink[h]) in the denominator, with no key and no value (scores are in units of log2 e)
     const float sink_log2 = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
     top = fmaxf(top, sink_log2);
     float denom = sink != nullptr ? exp2f(sink_log2 - top) : 0.0f;
-    for (int cc = c_first; cc <= c_last; cc++)
+    for (int cc = 0; cc <= c_last; cc++)
         denom += __ldcg(part_ml + (first + cc) * 2 + 1) * exp2f(__ldcg(part_ml + (first + cc) * 2) - top);
     // a gate per (token, head) opens the result by its sigmoid
     const float open = gate != nullptr ? 1.0f / (1.0f + __expf(-gate[(long)t * ld_gate + h])) : 1.0f;
-    for (int d = threadIdx.x; d < D; d += 128) {
+    for (int d = threadIdx.x; d < vdim; d += 128) {
         float o = 0.0f;
-        for (int cc = c_first; cc <= c_last; cc++)
+        for (int cc = 0; cc <= c_last; cc++)
             o += __ldcg(part_acc + (first + cc) * D + d) * exp2f(__ldcg(part_ml + (first + cc) * 2) - top);
-        out[(long)t * ld_out + (long)h * D + d] = __float2bfloat16_rn(o / denom * open);
+        out[(long)t * ld_out + (long)h * vdim + d] = __float2bfloat16_rn(o / denom * open);
     }
 }
 
@@ -395,6 +406,48 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
 // positions: block > 0, a query sees only keys of its own block, counted from position 0; with a gate:
 // fp32 [tokens, >= heads], head h's result times sigmoid(gate[t, h]); with a sink: fp32 [heads], exp(sink[h]) joins
 // head h's softmax denominator)
+// The widest form: key rows of `dim` and value rows of `vdim` entries (equal and one of 16, 32, 64, 128, 256, or
+// any multiples of 8 up to 256; the scratch's rows then have the least of those sizes that holds both), and the keys
+// below `keep` stay visible behind a window.  max_chunks * chunk covers the most keys a token of the step sees.
+extern "C" int mllm_decode_split_attention_kept(void* out, long ld_out, const void* q, long ld_q, const void* k_pages,
+                                                const void* v_pages, const int* block_table, int max_blocks,
+                                                const int* positions, const int* token_item, int n_tokens, int n_heads,
+                                                int n_kv_heads, int dim, int vdim, int page_size, float scale, float cap,
+                                                int window, int block, int keep, const float* gate, long ld_gate,
+                                                const float* sink, int chunk, int max_chunks, float* part_acc,
+                                                float* part_ml, int* counters, void* stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0)
+        return fail("split_attention: heads must be a multiple of key/value heads");
+    if (chunk <= 0 || max_chunks <= 0 || max_chunks > 65535 || n_heads > 65535)
+        return fail("split_attention: bad chunking");
+    if (ld_q % 8 != 0) return fail("split_attention: the row stride of q must be a multiple of 8");
+    if (keep < 0 || (keep > 0 && block > 0)) return fail("split_attention: kept first keys go with a window, not with blocks of positions");
+    if (dim <= 0 || vdim <= 0 || dim % 8 != 0 || vdim % 8 != 0 || dim > 256 || vdim > 256)
+        return fail("split_attention: key and value sizes are multiples of 8 up to 256");
+    const int most = dim > vdim ? dim : vdim;
+    const int size = most <= 16 ? 16 : (most <= 32 ? 32 : (most <= 64 ? 64 : (most <= 128 ? 128 : 256)));
+    const bool full = dim == size && vdim == size;
+    cudaStream_t s = (cudaStream_t)stream;
+    dim3 grid(n_tokens, n_heads, max_chunks);
+#define LAUNCH_SPLIT(D, FULL)                                                                                        \
+    launch_kernel(g_dependent_launch != 0, split_attention_kernel<D, FULL>, grid, dim3(128), 0, s, (bf16*)out, ld_out, \
+                  (const bf16*)q, ld_q, (const bf16*)k_pages, (const bf16*)v_pages, block_table, max_blocks,         \
+                  positions, token_item, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, block, keep, \
+                  gate, ld_gate, sink, chunk, max_chunks, part_acc, part_ml, counters)
+#define PICK_SPLIT(D) do { if (full) LAUNCH_SPLIT(D, true); else LAUNCH_SPLIT(D, false); } while (0)
+    switch (size) {
+    case 16: PICK_SPLIT(16); break;
+    case 32: PICK_SPLIT(32); break;
+    case 64: PICK_SPLIT(64); break;
+    case 128: PICK_SPLIT(128); break;
+    default: PICK_SPLIT(256); break;
+    }
+#undef PICK_SPLIT
+#undef LAUNCH_SPLIT
+    return check_launch("split_attention_kernel");
+}
+
 extern "C" int mllm_decode_split_attention_sink(void* out, long ld_out, const void* q, long ld_q, const void* k_pages,
                                                 const void* v_pages, const int* block_table, int max_blocks,
                                                 const int* positions, const int* token_item, int n_tokens, int n_heads,
@@ -402,29 +455,14 @@ extern "C" int mllm_decode_split_attention_sink(void* out, long ld_out, const vo
                                                 int window, int block, const float* gate, long ld_gate, const float* sink,
                                                 int chunk, int max_chunks, float* part_acc, float* part_ml, int* counters,
                                                 void* stream) {
-    if (n_tokens <= 0) return 0;
-    if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0)
-        return fail("split_attention: heads must be a multiple of key/value heads");
-    if (chunk <= 0 || max_chunks <= 0 || max_chunks > 65535 || n_heads > 65535)
-        return fail("split_attention: bad chunking");
-    if (ld_q % 8 != 0) return fail("split_attention: the row stride of q must be a multiple of 8");
-    cudaStream_t s = (cudaStream_t)stream;
-    dim3 grid(n_tokens, n_heads, max_chunks);
-#define LAUNCH_SPLIT(D)                                                                                              \
-    launch_kernel(g_dependent_launch != 0, split_attention_kernel<D>, grid, dim3(128), 0, s, (bf16*)out, ld_out,     \
-                  (const bf16*)q, ld_q, (const bf16*)k_pages, (const bf16*)v_pages, block_table, max_blocks,         \
-                  positions, token_item, n_heads, n_kv_heads, page_size, scale, cap, window, block, gate, ld_gate,   \
-                  sink, chunk, max_chunks, part_acc, part_ml, counters)
     switch (head_size) {
-    case 16: LAUNCH_SPLIT(16); break;
-    case 32: LAUNCH_SPLIT(32); break;
-    case 64: LAUNCH_SPLIT(64); break;
-    case 128: LAUNCH_SPLIT(128); break;
-    case 256: LAUNCH_SPLIT(256); break;
+    case 16: case 32: case 64: case 128: case 256: break;
     default: return fail("split_attention: head size must be 16, 32, 64, 128 or 256");
     }
-#undef LAUNCH_SPLIT
-    return check_launch("split_attention_kernel");
+    return mllm_decode_split_attention_kept(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions,
+                                            token_item, n_tokens, n_heads, n_kv_heads, head_size, head_size, page_size, scale,
+                                            cap, window, block, 0, gate, ld_gate, sink, chunk, max_chunks, part_acc, part_ml,
+                                            counters, stream);
 }
 
 extern "C" int mllm_decode_split_attention_masked(void* out, long ld_out, const void* q, long ld_q, const void* k_pages,

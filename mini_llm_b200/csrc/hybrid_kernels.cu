@@ -15,7 +15,7 @@
 //   head_norm_store   queries and keys divided by their root mean square per head (no gain), and the
 //                     keys and values into their cache pages
 // capped_attention also takes a chunked mask (a query sees the keys of its own block of `chunk`
-// positions only) and a gate per (token, head) whose sigmoid multiplies the head's result;
+// positions only), a number of first keys that stay visible behind a window, and a gate per (token, head) whose sigmoid multiplies the head's result;
 // linear_recurrence also takes a decay per key channel instead of one per head.
 // Every kernel is templated on the element type of the activations (float: the true 32-bit path;
 // bfloat16: the serving path) and is launched as a programmatic dependent of the kernel before it.
@@ -165,7 +165,7 @@ extern "C" int mllm_hybrid_head_norm_store(void* qkv, long ld, int k_off, int v_
 // ---------------------------------------------------------------------------
 // Causal attention with capped scores, one block per (token, head): the plain form, which takes
 // every size.  score = cap * tanh((q . k) * scale / cap) (cap <= 0: no cap); the query at position
-// p sees keys max(0, p - window + 1) .. p (window <= 0: all).  Four warps take the keys in turn,
+// p sees keys max(0, p - window + 1) .. p (window <= 0: all) and those below `keep`.  Four warps take the keys in turn,
 // each with an online softmax; their states are merged in a fixed order.
 // ---------------------------------------------------------------------------
 constexpr int CAP_MAX_HEAD = 256;
@@ -180,13 +180,22 @@ __device__ __forceinline__ int first_visible(int p, int window, int chunk) {
     return lo;
 }
 
+// Keys below `keep` stay visible to every query after them, whatever the window.  A tile walk over a run's keys
+// [0, keep) and [lo, p_last] starts at tile 0 if anything is kept and leaps from the kept tiles to the one that holds lo.
+__device__ __forceinline__ bool key_visible(int j, int lo, int keep) { return j >= lo || j < keep; }
+__device__ __forceinline__ int first_tile(int first_base, int keep) { return keep > 0 ? 0 : first_base; }
+__device__ __forceinline__ int next_tile(int base, int step, int first_base, int keep) {
+    base += step;
+    return base >= keep && base < first_base ? first_base : base;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 capped_attention_plain_kernel(T* __restrict__ out, long ld_out, const T* __restrict__ q, long ld_q,
                               const T* __restrict__ k_pages, const T* __restrict__ v_pages,
                               const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                               const int* __restrict__ token_item, int n_heads, int n_kv_heads, int dim, int vdim,
-                              int page_size, float scale, float cap, int window, int chunk,
+                              int page_size, float scale, float cap, int window, int chunk, int keep,
                               const float* __restrict__ gate, long ld_gate, const float* __restrict__ sink) {
     dependents_may_start();
     wait_for_earlier_kernels();
@@ -206,7 +215,9 @@ capped_attention_plain_kernel(T* __restrict__ out, long ld_out, const T* __restr
     }
     float m = -INFINITY, l = 0.0f;
     const int lo = first_visible(p, window, chunk);
-    for (int j = lo + warp; j <= p; j += 4) {
+    const int n_kept = min(keep, lo);                        // kept keys ahead of the window, then the window's
+    for (int i = warp; i <= p - lo + n_kept; i += 4) {
+        const int j = i < n_kept ? i : i - n_kept + lo;
         const long slot = (long)bt[j / page_size] * page_size + (j % page_size);
         const T* kr = k_pages + (slot * n_kv_heads + hk) * dim;
         const T* vr = v_pages + (slot * n_kv_heads + hk) * vdim;
@@ -287,7 +298,7 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
                               const T* __restrict__ k_pages, const T* __restrict__ v_pages,
                               const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                               const int* __restrict__ token_item, int n_tokens, int n_heads, int n_kv_heads, int dim,
-                              int vdim, int page_size, float scale, float cap, int window, int chunk,
+                              int vdim, int page_size, float scale, float cap, int window, int chunk, int keep,
                               const float* __restrict__ gate, long ld_gate, const float* __restrict__ sink,
                               int tokens_per_block, int heads_per_block) {
     dependents_may_start();
@@ -350,12 +361,12 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
 #pragma unroll
         for (int i = 0; i < MAXV; i++) {
             const int kp = base + key_row[i], vp = base + value_row[i];
-            if (key_row[i] >= 0 && kp <= p_last && kp >= p_lo) {
+            if (key_row[i] >= 0 && kp <= p_last && key_visible(kp, p_lo, keep)) {
                 const int block = page_shift >= 0 ? kp >> page_shift : kp / page_size;
                 const long slot = (long)bt[block] * page_size + (kp - block * page_size);
                 key_vec[i] = *reinterpret_cast<const uint4*>(k_pages + (slot * n_kv_heads + hk) * dim + key_col[i]);
             }
-            if (value_row[i] >= 0 && vp <= p_last && vp >= p_lo) {
+            if (value_row[i] >= 0 && vp <= p_last && key_visible(vp, p_lo, keep)) {
                 const int block = page_shift >= 0 ? vp >> page_shift : vp / page_size;
                 const long slot = (long)bt[block] * page_size + (vp - block * page_size);
                 value_vec[i] = *reinterpret_cast<const uint4*>(v_pages + (slot * n_kv_heads + hk) * vdim + value_col[i]);
@@ -374,8 +385,10 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
         const int lo = first_visible(p_first, window, chunk);
         const int* bt = block_table + (long)item * max_blocks;
         const int first_base = (lo / TILE_KEYS) * TILE_KEYS;
-        fetch(bt, first_base, p_last, lo);          // (pages before the first visible key may be gone)
-        for (int base = first_base; base <= p_last; base += TILE_KEYS) {
+        int base = first_tile(first_base, keep), next = 0;
+        fetch(bt, base, p_last, lo);                // (pages before the first visible key may be gone)
+        for (; base <= p_last; base = next) {
+            next = next_tile(base, TILE_KEYS, first_base, keep);
             __syncthreads();                                  // the block before has been read; q_rows are written
             const int n_keys = min(TILE_KEYS, p_last + 1 - base);
 #pragma unroll
@@ -385,14 +398,14 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
             }
             __syncthreads();
             // the next block's rows are asked for now and arrive while this one is worked on
-            if (base + TILE_KEYS <= p_last) fetch(bt, base + TILE_KEYS, p_last, lo);
+            if (next <= p_last) fetch(bt, next, p_last, lo);
             // which of the warp's rows see a key of this block at all
             bool any = false, seen[R];
             int first_seen[R];
 #pragma unroll
             for (int s = 0; s < R; s++) {
                 first_seen[s] = first_visible(row_pos[s], window, chunk);
-                seen[s] = row_item[s] == item && base <= row_pos[s] && base + TILE_KEYS > first_seen[s];
+                seen[s] = row_item[s] == item && base <= row_pos[s] && (base + TILE_KEYS > first_seen[s] || base < keep);
                 any = any || seen[s];
             }
             if (!any) continue;                               // (uniform in the warp; the barriers are at the loop's head)
@@ -416,7 +429,7 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
             const int pos = base + lane;
 #pragma unroll
             for (int s = 0; s < R; s++) {
-                const bool mine = seen[s] && lane < n_keys && pos <= row_pos[s] && pos >= first_seen[s];
+                const bool mine = seen[s] && lane < n_keys && pos <= row_pos[s] && key_visible(pos, first_seen[s], keep);
                 const float score = mine ? capped(dot[s] * scale, cap, inv_cap) : -INFINITY;
                 const float block_max = warp_max(score);
                 float rescale = 1.0f, e = 0.0f;
@@ -477,8 +490,8 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
 }
 
 // ---------------------------------------------------------------------------
-// The same attention as register tiles, for the common sizes (values of 64 or 128 entries, keys of up to 128,
-// no gate, no mask of blocks).  A block of 256 threads takes 64 (token, head) rows of one key/value head and walks
+// The same attention as register tiles, for the common sizes (keys and values of up to 128 entries, no gate, no
+// mask of blocks).  A block of 256 threads takes 64 (token, head) rows of one key/value head and walks
 // the keys 64 at a time.  Thread (ty, tx) of a 16 x 16 grid holds the scores of rows 4 ty .. 4 ty + 3 against keys
 // tx, tx + 16, tx + 32, tx + 48 (sixteen sums, fed by 16-byte reads of q and k rows along the head: eight FMAs a
 // read), then, after the block's softmax step, the sums of those rows' values for columns 4 tx .. 4 tx + 3 (and
@@ -491,14 +504,14 @@ constexpr int BLOCK_ROWS = 64, BLOCK_KEYS = 64;
 constexpr int BLOCK_RT = 4;                                   // rows a thread (eight measured slower: 255 registers, one block fewer an SM)
 constexpr int BLOCK_THREADS = 16 * BLOCK_ROWS / BLOCK_RT;
 
-template <typename T, int VG>          // VG: 64-entry groups of a value (1 or 2)
+template <typename T, int VG>          // VG: 64-entry groups that hold a value (1 or 2; the last may be filled in part)
 __global__ void __launch_bounds__(BLOCK_THREADS)
 capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restrict__ q, long ld_q,
                               const T* __restrict__ k_pages, const T* __restrict__ v_pages,
                               const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                               const int* __restrict__ token_item, int n_tokens, int n_heads, int n_kv_heads, int dim,
-                              int page_size, float scale, float cap, int window, const float* __restrict__ sink,
-                              int tokens_per_block, int heads_per_block) {
+                              int vdim, int page_size, float scale, float cap, int window, int keep,
+                              const float* __restrict__ sink, int tokens_per_block, int heads_per_block) {
     dependents_may_start();
     wait_for_earlier_kernels();
     constexpr int VDIM = 64 * VG;
@@ -566,7 +579,7 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
     for (int i = 0; i < MAXV; i++) {
         const int u = tid + i * BLOCK_THREADS;
         value_row[i] = u / (VDIM / VEC);
-        value_col[i] = (u % (VDIM / VEC)) * VEC;
+        value_col[i] = (u % (VDIM / VEC)) * VEC;             // (columns from vdim on stay zero)
         value_vec[i] = make_uint4(0u, 0u, 0u, 0u);
     }
     auto fetch = [&](const int* bt, int base, int p_last, int p_lo) {
@@ -574,7 +587,7 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
         for (int i = 0; i < MAXK; i++) {
             const int kp = base + key_row[i];
             key_vec[i] = make_uint4(0u, 0u, 0u, 0u);
-            if (key_row[i] >= 0 && kp <= p_last && kp >= p_lo) {          // (pages before the first visible key may be gone)
+            if (key_row[i] >= 0 && kp <= p_last && key_visible(kp, p_lo, keep)) {      // (pages before the first visible key may be gone)
                 const int block = page_shift >= 0 ? kp >> page_shift : kp / page_size;
                 const long slot = (long)bt[block] * page_size + (kp - block * page_size);
                 key_vec[i] = *reinterpret_cast<const uint4*>(k_pages + (slot * n_kv_heads + hk) * dim + key_col[i]);
@@ -584,10 +597,10 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
         for (int i = 0; i < MAXV; i++) {
             const int vp = base + value_row[i];
             value_vec[i] = make_uint4(0u, 0u, 0u, 0u);
-            if (vp <= p_last && vp >= p_lo) {
+            if (value_col[i] < vdim && vp <= p_last && key_visible(vp, p_lo, keep)) {
                 const int block = page_shift >= 0 ? vp >> page_shift : vp / page_size;
                 const long slot = (long)bt[block] * page_size + (vp - block * page_size);
-                value_vec[i] = *reinterpret_cast<const uint4*>(v_pages + (slot * n_kv_heads + hk) * VDIM + value_col[i]);
+                value_vec[i] = *reinterpret_cast<const uint4*>(v_pages + (slot * n_kv_heads + hk) * vdim + value_col[i]);
             }
         }
     };
@@ -601,8 +614,10 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
         const int lo = first_visible(p_first, window, 0);
         const int* bt = block_table + (long)item * max_blocks;
         const int first_base = (lo / BLOCK_KEYS) * BLOCK_KEYS;
-        fetch(bt, first_base, p_last, lo);
-        for (int base = first_base; base <= p_last; base += BLOCK_KEYS) {
+        int base = first_tile(first_base, keep), next = 0;
+        fetch(bt, base, p_last, lo);
+        for (; base <= p_last; base = next) {
+            next = next_tile(base, BLOCK_KEYS, first_base, keep);
             __syncthreads();                                  // the tile before has been read
 #pragma unroll
             for (int i = 0; i < MAXK; i++)
@@ -611,12 +626,12 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
             for (int i = 0; i < MAXV; i++) widen<T>(value_vec[i], values + value_row[i] * vd + value_col[i]);
             __syncthreads();
             // the next tile's rows are asked for now and arrive while this one is worked on
-            if (base + BLOCK_KEYS <= p_last) fetch(bt, base + BLOCK_KEYS, p_last, lo);
+            if (next <= p_last) fetch(bt, next, p_last, lo);
             // does any row of this warp see a key of this tile?
             bool any = false;
 #pragma unroll
             for (int i = 0; i < RT; i++)
-                any = any || (my_item[i] == item && base <= my_pos[i] && base + BLOCK_KEYS > my_first[i]);
+                any = any || (my_item[i] == item && base <= my_pos[i] && (base + BLOCK_KEYS > my_first[i] || base < keep));
             if (!__any_sync(0xffffffffu, any)) continue;      // (uniform in the warp; the barriers are at the loop's head)
             float acc[RT][4];
 #pragma unroll
@@ -647,7 +662,7 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     const int pos = base + tx + 16 * j;
-                    const bool seen = row_here && pos <= my_pos[i] && pos >= my_first[i];
+                    const bool seen = row_here && pos <= my_pos[i] && key_visible(pos, my_first[i], keep);
                     score[j] = seen ? capped(acc[i][j] * scale, cap, inv_cap) : -INFINITY;
                     top = fmaxf(top, score[j]);
                 }
@@ -714,7 +729,8 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
         for (int g = 0; g < VG; g++)
 #pragma unroll
             for (int c = 0; c < 4; c++)
-                out[(long)token * ld_out + (long)head * VDIM + 64 * g + tx * 4 + c] = from_f32<T>(o[i][4 * g + c] * inv);
+                if (64 * g + tx * 4 + c < vdim)
+                    out[(long)token * ld_out + (long)head * vdim + 64 * g + tx * 4 + c] = from_f32<T>(o[i][4 * g + c] * inv);
     }
 }
 
@@ -723,16 +739,16 @@ static size_t capped_block_shared(int dim, int vdim) {
            sizeof(int) * 2 * BLOCK_ROWS;
 }
 
-// (keys in whole 16-byte vectors, values of 64 or 128 entries)
+// (keys and values in whole 16-byte vectors; values narrower than half their groups go to the tiles of few rows)
 static bool capped_block_takes(int dim, int vdim, int vec) {
-    return dim > 0 && dim <= 128 && dim % vec == 0 && dim % 4 == 0 && (vdim == 64 || vdim == 128);
+    return dim > 0 && dim <= 128 && dim % vec == 0 && dim % 4 == 0 && vdim > 32 && vdim <= 128 && vdim % vec == 0 && vdim % 4 == 0;
 }
 
 template <typename T, int VG>
 static int launch_capped_block(void* out, long ld_out, const void* q, long ld_q, const void* k_pages, const void* v_pages,
                                const int* block_table, int max_blocks, const int* positions, const int* token_item, int n_tokens,
-                               int n_heads, int n_kv_heads, int dim, int page_size, float scale, float cap, int window,
-                               const float* sink, cudaStream_t s) {
+                               int n_heads, int n_kv_heads, int dim, int vdim, int page_size, float scale, float cap, int window,
+                               int keep, const float* sink, cudaStream_t s) {
     const int group = n_heads / n_kv_heads;
     const int heads_per_block = group < BLOCK_ROWS ? group : BLOCK_ROWS;
     const int tokens_per_block = BLOCK_ROWS / heads_per_block;
@@ -744,7 +760,7 @@ static int launch_capped_block(void* out, long ld_out, const void* q, long ld_q,
     dim3 grid((n_tokens + tokens_per_block - 1) / tokens_per_block, n_kv_heads * chunks);
     launch_kernel(g_dependent_launch != 0, capped_attention_block_kernel<T, VG>, grid, dim3(BLOCK_THREADS), shared, s, (T*)out, ld_out, (const T*)q,
                   ld_q, (const T*)k_pages, (const T*)v_pages, block_table, max_blocks, positions, token_item, n_tokens, n_heads,
-                  n_kv_heads, dim, page_size, scale, cap, window, sink, tokens_per_block, heads_per_block);
+                  n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, sink, tokens_per_block, heads_per_block);
     return check_launch("capped_attention_block_kernel");
 }
 
@@ -763,7 +779,7 @@ template <typename T, int R, int SIZE>
 static int launch_capped_tiles(void* out, long ld_out, const void* q, long ld_q, const void* k_pages, const void* v_pages,
                                const int* block_table, int max_blocks, const int* positions, const int* token_item, int n_tokens,
                                int n_heads, int n_kv_heads, int dim, int vdim, int page_size, float scale, float cap, int window,
-                               int chunk, const float* gate, long ld_gate, const float* sink, cudaStream_t s) {
+                               int chunk, int keep, const float* gate, long ld_gate, const float* sink, cudaStream_t s) {
     constexpr int ROWS = TILE_WARPS * R;
     const int group = n_heads / n_kv_heads;
     const int heads_per_block = group < ROWS ? group : ROWS;
@@ -777,7 +793,7 @@ static int launch_capped_tiles(void* out, long ld_out, const void* q, long ld_q,
     dim3 grid((n_tokens + tokens_per_block - 1) / tokens_per_block, n_kv_heads * chunks);
     launch_kernel(g_dependent_launch != 0, capped_attention_tiled_kernel<T, R, SIZE>, grid, dim3(TILE_WARPS * 32), shared, s, (T*)out,
                   ld_out, (const T*)q, ld_q, (const T*)k_pages, (const T*)v_pages, block_table, max_blocks, positions, token_item,
-                  n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, gate, ld_gate, sink,
+                  n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, sink,
                   tokens_per_block, heads_per_block);
     return check_launch("capped_attention_tiled_kernel");
 }
@@ -786,22 +802,22 @@ template <typename T>
 static int launch_capped_attention(bool tiled, void* out, long ld_out, const void* q, long ld_q, const void* k_pages,
                                    const void* v_pages, const int* block_table, int max_blocks, const int* positions,
                                    const int* token_item, int n_tokens, int n_heads, int n_kv_heads, int dim, int vdim,
-                                   int page_size, float scale, float cap, int window, int chunk, const float* gate, long ld_gate,
-                                   const float* sink, cudaStream_t s) {
+                                   int page_size, float scale, float cap, int window, int chunk, int keep, const float* gate,
+                                   long ld_gate, const float* sink, cudaStream_t s) {
     if (!tiled) {
         launch_kernel(g_dependent_launch != 0, capped_attention_plain_kernel<T>, dim3(n_tokens, n_heads), dim3(128), 0, s, (T*)out,
                       ld_out, (const T*)q, ld_q, (const T*)k_pages, (const T*)v_pages, block_table, max_blocks, positions,
-                      token_item, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, gate, ld_gate, sink);
+                      token_item, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, sink);
         return check_launch("capped_attention_plain_kernel");
     }
     // the common sizes go to the register tiles
     if (gate == nullptr && chunk == 0 && n_tokens * (long)n_heads >= 2048 && capped_block_takes(dim, vdim, 16 / (int)sizeof(T)) &&
         (ld_q * sizeof(T)) % 16 == 0) {
-        if (vdim == 64)
+        if (vdim <= 64)
             return launch_capped_block<T, 1>(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions, token_item,
-                                             n_tokens, n_heads, n_kv_heads, dim, page_size, scale, cap, window, sink, s);
+                                             n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, sink, s);
         return launch_capped_block<T, 2>(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions, token_item,
-                                         n_tokens, n_heads, n_kv_heads, dim, page_size, scale, cap, window, sink, s);
+                                         n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, sink, s);
     }
     // rows a warp: four where the step has rows enough for the blocks to fill the GPU all the same
     // (and their shared memory fits), else two
@@ -810,7 +826,7 @@ static int launch_capped_attention(bool tiled, void* out, long ld_out, const voi
     if (capped_tiled_shared(dim, vdim, per_warp) > 160 * 1024) per_warp = 2;
 #define TILES(R, SIZE)                                                                                                        \
     return launch_capped_tiles<T, R, SIZE>(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions, token_item, \
-                                           n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, gate, ld_gate, sink, s)
+                                           n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, sink, s)
     const int size = (dim > vdim ? dim : vdim) <= 64 ? 64 : ((dim > vdim ? dim : vdim) <= 128 ? 128 : 256);
     if (per_warp == 4) { if (size == 64) TILES(4, 64); if (size == 128) TILES(4, 128); TILES(4, 256); }
     if (size == 64) TILES(2, 64);
@@ -822,22 +838,23 @@ static int launch_capped_attention(bool tiled, void* out, long ld_out, const voi
 extern "C" int mllm_hybrid_capped_attention(void* out, long ld_out, const void* q, long ld_q, const void* k_pages,
                                             const void* v_pages, const int* block_table, int max_blocks, const int* positions,
                                             const int* token_item, int n_tokens, int n_heads, int n_kv_heads, int dim, int vdim,
-                                            int page_size, float scale, float cap, int window, int chunk, const float* gate,
+                                            int page_size, float scale, float cap, int window, int chunk, int keep, const float* gate,
                                             long ld_gate, const float* sink, int tiled, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     if (dim <= 0 || dim > CAP_MAX_HEAD || vdim <= 0 || vdim > CAP_MAX_HEAD) return fail("capped_attention: key and value sizes must be in 1..256");
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return fail("capped_attention: heads must be a multiple of the key/value heads");
     if (n_heads > 65535) return fail("capped_attention: too many heads for one launch");
+    if (keep < 0 || (keep > 0 && chunk > 0)) return fail("capped_attention: kept first keys go with a window, not with blocks of positions");
     if (tiled && !mllm_hybrid_capped_attention_tiled_takes(dim, vdim, dtype == DT_F32 ? 4 : 8)) return fail("capped_attention: the tiles do not take these sizes");
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == DT_F32)
         return launch_capped_attention<float>(tiled != 0, out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions,
-                                              token_item, n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, gate,
-                                              ld_gate, sink, s);
+                                              token_item, n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep,
+                                              gate, ld_gate, sink, s);
     if (dtype == DT_BF16)
         return launch_capped_attention<bf16>(tiled != 0, out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions,
-                                             token_item, n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, gate,
-                                             ld_gate, sink, s);
+                                             token_item, n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep,
+                                             gate, ld_gate, sink, s);
     return fail("capped_attention: unknown dtype");
 }
 
@@ -1177,9 +1194,13 @@ extern "C" int mllm_hybrid_linear_recurrence(const RecurrenceParams* params, int
 //                largest s (the lower index wins a tie) with s as the weight of their INPUT; if
 //                there is a shared expert, one more pair: expert `n_experts`, input weight 1,
 //                output weight sigmoid(w_shared_gate . x) (or 1 for a shared expert without a gate).
-//                With `softmax_of_chosen`: z (+ a bias per expert) itself ranks the experts, the
+//                ROUTE_SOFTMAX_OF_CHOSEN: z (+ a bias per expert) itself ranks the experts, the
 //                chosen ones' OUTPUTS are weighed by the softmax over the chosen logits only, and
-//                their inputs by 1
+//                their inputs by 1.  ROUTE_SOFTMAX_OF_ALL: s = the softmax over all outputs; s plus a
+//                correction per output ranks them, the chosen ones' outputs are weighed by s over
+//                the chosen ones' sum (+ 1e-20), times `scale`.  The last `n_identity` outputs are
+//                identity experts, whose output is the token itself: such a choice becomes -1 and
+//                its weight goes into the token's identity weight
 //   expert_up    act[pair, f] = silu(W_gate[e] x') * (W_up[e] x') with x' = weight * x
 //   expert_down  hidden[t] += sum over the token's pairs of out_weight * W_down[e] act[pair] (or, with `assign`,
 //                hidden[t] = that sum)
@@ -1216,64 +1237,118 @@ template <> struct Vec16<bf16> {
 __device__ __forceinline__ bool aligned16(const void* p) { return (reinterpret_cast<unsigned long long>(p) & 15ull) == 0; }
 static bool aligned_host(const void* p) { return (reinterpret_cast<unsigned long long>(p) & 15ull) == 0; }
 
+// How a token's experts are chosen and weighed (the launcher's `rule`).
+enum RouteRule { ROUTE_SIGMOID_ON_INPUT = 0, ROUTE_SOFTMAX_OF_CHOSEN = 1, ROUTE_SOFTMAX_OF_ALL = 2 };
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, const float* __restrict__ router_bias,
-             const T* __restrict__ shared_gate, int shared_plain, int softmax_of_chosen, int width, int n_experts, int top,
-             int pairs, int* __restrict__ choice, float* __restrict__ in_weight, float* __restrict__ out_weight) {
+             const float* __restrict__ correction, const T* __restrict__ shared_gate, int shared_plain, int rule, float scale,
+             int width, int n_outputs, int n_identity, int top, int pairs, int* __restrict__ choice,
+             float* __restrict__ in_weight, float* __restrict__ out_weight, float* __restrict__ identity_weight) {
     dependents_may_start();
     wait_for_earlier_kernels();
     extern __shared__ float shared[];
     float* row = shared;                       // [width]
-    float* score = row + width;                // [n_experts + 1]
+    float* score = row + width;                // [n_outputs + 1]: what ranks the experts
+    float* share = score + n_outputs + 1;      // [n_outputs]: the softmax over all outputs (ROUTE_SOFTMAX_OF_ALL)
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int c = threadIdx.x; c < width; c += blockDim.x) row[c] = to_f32(x[(long)t * ld_x + c]);
     __syncthreads();
-    for (int e = warp; e < n_experts + (shared_gate != nullptr ? 1 : 0); e += 4) {
-        const T* w = e < n_experts ? router + (long)e * width : shared_gate;
+    for (int e = warp; e < n_outputs + (shared_gate != nullptr ? 1 : 0); e += 4) {
+        const T* w = e < n_outputs ? router + (long)e * width : shared_gate;
         float z = 0.0f;
-        for (int c = lane; c < width; c += 32) z = fmaf(to_f32(w[c]), row[c], z);
+        constexpr int N = Vec16<T>::N;
+        if (width % N == 0 && aligned16(w)) {
+            for (int c = lane * N; c < width; c += 32 * N) {
+                float a[N];
+                Vec16<T>::load(w + c, a);
+#pragma unroll
+                for (int i = 0; i < N; i++) z = fmaf(a[i], row[c + i], z);
+            }
+        } else {
+            for (int c = lane; c < width; c += 32) z = fmaf(to_f32(w[c]), row[c], z);
+        }
         z = warp_sum(z);
-        if (e < n_experts && router_bias != nullptr) z += router_bias[e];
-        // (the chosen logits' softmax needs the logits themselves)
-        if (lane == 0) score[e] = softmax_of_chosen && e < n_experts ? z : sigmoid_f(z);
+        if (e < n_outputs && router_bias != nullptr) z += router_bias[e];
+        // (a softmax needs the logits themselves)
+        if (lane == 0) score[e] = rule != ROUTE_SIGMOID_ON_INPUT && e < n_outputs ? z : sigmoid_f(z);
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
-        float largest = 0.0f, total = 0.0f;
-        for (int k = 0; k < top; k++) {
-            int best = -1;
-            float best_score = -INFINITY;
-            for (int e = 0; e < n_experts; e++)
-                if (score[e] > best_score) best = e, best_score = score[e];
-            if (best < 0) best = 0, best_score = score[0];      // (scores that are no numbers)
-            choice[(long)t * pairs + k] = best;
-            if (softmax_of_chosen) {
-                // weights of the outputs: the softmax over the chosen logits only (the first is the largest)
-                if (k == 0) largest = best_score;
-                const float e = expf(best_score - largest);
-                in_weight[(long)t * pairs + k] = 1.0f;
-                out_weight[(long)t * pairs + k] = e;
-                total += e;
-            } else {
-                in_weight[(long)t * pairs + k] = best_score;
-                out_weight[(long)t * pairs + k] = 1.0f;
-            }
+    if (warp != 0) return;
+    // one warp ranks: lane l looks at outputs l, l + 32, ...
+    if (rule == ROUTE_SOFTMAX_OF_ALL) {
+        float most = -INFINITY, sum = 0.0f;
+        for (int e = lane; e < n_outputs; e += 32) most = fmaxf(most, score[e]);
+        most = warp_max(most);
+        for (int e = lane; e < n_outputs; e += 32) {
+            share[e] = expf(score[e] - most);
+            sum += share[e];
+        }
+        sum = warp_sum(sum);
+        for (int e = lane; e < n_outputs; e += 32) {
+            share[e] /= sum;
+            score[e] = share[e] + (correction != nullptr ? correction[e] : 0.0f);
+        }
+        __syncwarp();
+    }
+    const int n_real = n_outputs - n_identity;
+    float largest = 0.0f, total = 0.0f;
+    for (int k = 0; k < top; k++) {
+        int best = n_outputs;
+        float best_score = -INFINITY;
+        for (int e = lane; e < n_outputs; e += 32)
+            if (score[e] > best_score) best = e, best_score = score[e];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float other_score = __shfl_xor_sync(0xffffffffu, best_score, o);
+            const int other = __shfl_xor_sync(0xffffffffu, best, o);
+            if (other_score > best_score || (other_score == best_score && other < best)) best = other, best_score = other_score;
+        }
+        if (best >= n_outputs) best = 0, best_score = score[0];      // (scores that are no numbers)
+        if (k == 0) largest = best_score;                            // (the first is the largest)
+        float weight = best_score;
+        if (rule == ROUTE_SOFTMAX_OF_CHOSEN) weight = expf(best_score - largest);
+        if (rule == ROUTE_SOFTMAX_OF_ALL) weight = share[best];
+        total += weight;
+        if (lane == 0) {
+            const long pair = (long)t * pairs + k;
+            choice[pair] = best;
+            in_weight[pair] = rule == ROUTE_SIGMOID_ON_INPUT ? weight : 1.0f;
+            out_weight[pair] = rule == ROUTE_SIGMOID_ON_INPUT ? 1.0f : weight;
             score[best] = -INFINITY;
         }
-        if (softmax_of_chosen)
-            for (int k = 0; k < top; k++) out_weight[(long)t * pairs + k] /= total;
-        if (shared_gate != nullptr || shared_plain) {
-            choice[(long)t * pairs + top] = n_experts;
-            in_weight[(long)t * pairs + top] = 1.0f;
-            out_weight[(long)t * pairs + top] = shared_gate != nullptr ? score[n_experts] : 1.0f;
+        __syncwarp();
+    }
+    if (lane != 0) return;
+    if (rule != ROUTE_SIGMOID_ON_INPUT) {
+        // the chosen experts' weights over their own sum; an identity expert's goes to the token's input itself
+        float passed = 0.0f;
+        for (int k = 0; k < top; k++) {
+            const long pair = (long)t * pairs + k;
+            const float weight = rule == ROUTE_SOFTMAX_OF_ALL ? out_weight[pair] / (total + 1e-20f) * scale : out_weight[pair] / total;
+            const bool identity = choice[pair] >= n_real;
+            if (identity) passed += weight, choice[pair] = -1;
+            out_weight[pair] = identity ? 0.0f : weight;
         }
+        if (identity_weight != nullptr) identity_weight[t] = passed;
+    }
+    if (shared_gate != nullptr || shared_plain) {
+        choice[(long)t * pairs + top] = n_real;
+        in_weight[(long)t * pairs + top] = 1.0f;
+        out_weight[(long)t * pairs + top] = shared_gate != nullptr ? score[n_outputs] : 1.0f;
     }
 }
 
 constexpr int UP_FEATURES = 32;                // inner features a block of expert_up takes (four a warp)
 
-template <typename T>
+// What an expert applies between its two products: silu(gate) * up, or (no gate matrix) the square of relu(up).
+__device__ __forceinline__ float relu_squared(float z) {
+    const float r = fmaxf(z, 0.0f);
+    return r * r;
+}
+
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long ld_x, const int* __restrict__ choice,
                  const float* __restrict__ in_weight, const long long* __restrict__ gate_of, const long long* __restrict__ up_of,
@@ -1283,6 +1358,7 @@ expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long
     extern __shared__ float row[];             // [width]: the token times its weight, rounded as an activation
     const int pair = blockIdx.x, t = pair / pairs;
     const int e = choice[pair];
+    if (e < 0) return;                         // (an identity expert: expert_down passes the input on)
     const int inner = inner_of[e];
     const int first = blockIdx.y * UP_FEATURES;
     if (first >= inner) return;
@@ -1290,8 +1366,8 @@ expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long
     for (int c = threadIdx.x; c < width; c += blockDim.x)
         row[c] = to_f32(from_f32<T>(weight * to_f32(x[(long)t * ld_x + c])));
     __syncthreads();
-    const T* gate = (const T*)gate_of[e];
     const T* up = (const T*)up_of[e];
+    const T* gate = GATED ? (const T*)gate_of[e] : up;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int f = first + warp; f < min(first + UP_FEATURES, inner); f += 8) {
         const T* g = gate + (long)f * width;
@@ -1301,19 +1377,23 @@ expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long
         if (width % N == 0 && aligned16(g) && aligned16(u)) {
             for (int c = lane * N; c < width; c += 32 * N) {
                 float a[N], b[N];
-                Vec16<T>::load(g + c, a);
+                if (GATED) Vec16<T>::load(g + c, a);
                 Vec16<T>::load(u + c, b);
 #pragma unroll
-                for (int i = 0; i < N; i++) zg = fmaf(a[i], row[c + i], zg), zu = fmaf(b[i], row[c + i], zu);
+                for (int i = 0; i < N; i++) {
+                    if (GATED) zg = fmaf(a[i], row[c + i], zg);
+                    zu = fmaf(b[i], row[c + i], zu);
+                }
             }
         } else {
             for (int c = lane; c < width; c += 32) {
-                zg = fmaf(to_f32(g[c]), row[c], zg);
+                if (GATED) zg = fmaf(to_f32(g[c]), row[c], zg);
                 zu = fmaf(to_f32(u[c]), row[c], zu);
             }
         }
-        zg = warp_sum(zg), zu = warp_sum(zu);
-        if (lane == 0) act[(long)pair * ld_act + f] = from_f32<T>(silu_f(zg) * zu);
+        if (GATED) zg = warp_sum(zg);
+        zu = warp_sum(zu);
+        if (lane == 0) act[(long)pair * ld_act + f] = from_f32<T>(GATED ? silu_f(zg) * zu : relu_squared(zu));
     }
 }
 
@@ -1321,7 +1401,8 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 expert_down_kernel(float* __restrict__ hidden, long ld_hidden, const T* __restrict__ act, long ld_act,
                    const int* __restrict__ choice, const float* __restrict__ out_weight, const long long* __restrict__ down_of,
-                   const int* __restrict__ inner_of, long ld_down, int width, int pairs, int assign) {
+                   const int* __restrict__ inner_of, long ld_down, int width, int pairs, int assign, const T* __restrict__ x,
+                   long ld_x, const float* __restrict__ identity_weight) {
     dependents_may_start();
     wait_for_earlier_kernels();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1330,6 +1411,7 @@ expert_down_kernel(float* __restrict__ hidden, long ld_hidden, const T* __restri
         for (int k = 0; k < pairs; k++) {
             const long pair = (long)t * pairs + k;
             const int e = choice[pair];
+            if (e < 0) continue;
             const int inner = inner_of[e];
             const T* w = (const T*)down_of[e] + (long)c * ld_down;
             const T* a = act + pair * ld_act;
@@ -1348,6 +1430,8 @@ expert_down_kernel(float* __restrict__ hidden, long ld_hidden, const T* __restri
             }
             total = fmaf(out_weight[pair], warp_sum(z), total);
         }
+        // identity experts hand the token on as it came
+        if (identity_weight != nullptr) total = fmaf(identity_weight[t], to_f32(x[(long)t * ld_x + c]), total);
         if (lane == 0) hidden[(long)t * ld_hidden + c] = assign ? total : hidden[(long)t * ld_hidden + c] + total;
     }
 }
@@ -1358,11 +1442,15 @@ expert_down_kernel(float* __restrict__ hidden, long ld_hidden, const T* __restri
 // (VEC: a thread takes the 16 bytes of columns that lie side by side, all of one expert: inner sizes that are
 // multiples of a vector's elements.  The token's weights per expert lie in shared memory, 0 for an expert it
 // did not choose, whose columns are written as zeros without reading the products.)
-template <typename T, bool VEC>
+// (GATED false: experts without a gate matrix; gu holds the ups alone, [T, total], and act is the square of relu.
+// With `identity_weight` the block's share of the token's columns of `hidden` also gets identity_weight[t] * x[t]:
+// set to it with `assign`, else added.)
+template <typename T, bool VEC, bool GATED>
 __global__ void __launch_bounds__(256)
 expert_combine_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ gu, long ld_gu, const int* __restrict__ choice,
                       const float* __restrict__ in_weight, const float* __restrict__ out_weight, int n_experts, int inner,
-                      int total, int top, int pairs) {
+                      int total, int top, int pairs, float* __restrict__ hidden, long ld_hidden, const T* __restrict__ x,
+                      long ld_x, const float* __restrict__ identity_weight, int width, int assign) {
     dependents_may_start();
     wait_for_earlier_kernels();
     extern __shared__ float weights[];             // [n_experts + 1][2]: input weight, output weight
@@ -1389,23 +1477,36 @@ expert_combine_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ gu
             if (s != 0.0f) {
                 float g[N], u[N];
                 Vec16<T>::load(row + c, g);
-                Vec16<T>::load(row + total + c, u);
+                if (GATED) Vec16<T>::load(row + total + c, u);
                 T* lanes = reinterpret_cast<T*>(&packed);
 #pragma unroll
-                for (int i = 0; i < N; i++) lanes[i] = from_f32<T>(silu_f(s * g[i]) * (s * u[i]) * o);
+                for (int i = 0; i < N; i++)
+                    lanes[i] = from_f32<T>(GATED ? silu_f(s * g[i]) * (s * u[i]) * o : relu_squared(s * g[i]) * o);
             }
             *reinterpret_cast<uint4*>(dst + c) = packed;
         } else {
             float v = 0.0f;
-            if (s != 0.0f) v = silu_f(s * to_f32(row[c])) * (s * to_f32(row[total + c])) * o;
+            if (s != 0.0f && GATED) v = silu_f(s * to_f32(row[c])) * (s * to_f32(row[total + c])) * o;
+            if (s != 0.0f && !GATED) v = relu_squared(s * to_f32(row[c])) * o;
             dst[c] = from_f32<T>(v);
         }
+    }
+    if (identity_weight != nullptr) {
+        const float passed = identity_weight[t];
+        if (assign || passed != 0.0f)
+            for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
+                const float v = passed * to_f32(x[(long)t * ld_x + c]);
+                float* h = hidden + (long)t * ld_hidden + c;
+                *h = assign ? v : *h + v;
+            }
     }
 }
 
 extern "C" int mllm_hybrid_expert_combine(void* act, long ld_act, const void* gu, long ld_gu, const int* choice,
                                           const float* in_weight, const float* out_weight, int n_experts, int inner, int total,
-                                          int top, int pairs, int n_tokens, int dtype, void* stream) {
+                                          int top, int pairs, int gated, float* hidden, long ld_hidden, const void* x, long ld_x,
+                                          const float* identity_weight, int width, int assign, int n_tokens, int dtype,
+                                          void* stream) {
     if (n_tokens <= 0) return 0;
     if (dtype != DT_F32 && dtype != DT_BF16) return fail("expert_combine: unknown dtype");
     cudaStream_t s = (cudaStream_t)stream;
@@ -1417,43 +1518,54 @@ extern "C" int mllm_hybrid_expert_combine(void* act, long ld_act, const void* gu
     dim3 grid(n_tokens, y);
     const size_t shared = sizeof(float) * 2 * ((size_t)n_experts + 1);
     if (shared > 48 * 1024) return fail("expert_combine: too many experts for the table of weights");
-#define RUN(T, VEC)                                                                                                             \
-    launch_kernel(g_dependent_launch != 0, expert_combine_kernel<T, VEC>, grid, dim3(256), shared, s, (T*)act, ld_act, (const T*)gu, \
-                  ld_gu, choice, in_weight, out_weight, n_experts, inner, total, top, pairs)
-    if (dtype == DT_F32) { if (vec) RUN(float, true); else RUN(float, false); }
-    else { if (vec) RUN(bf16, true); else RUN(bf16, false); }
+#define RUN(T, VEC, GATED)                                                                                                      \
+    launch_kernel(g_dependent_launch != 0, expert_combine_kernel<T, VEC, GATED>, grid, dim3(256), shared, s, (T*)act, ld_act,   \
+                  (const T*)gu, ld_gu, choice, in_weight, out_weight, n_experts, inner, total, top, pairs, hidden, ld_hidden,    \
+                  (const T*)x, ld_x, identity_weight, width, assign)
+#define RUN_AS(T)                                                                                                               \
+    do {                                                                                                                        \
+        if (vec) { if (gated) RUN(T, true, true); else RUN(T, true, false); }                                                   \
+        else { if (gated) RUN(T, false, true); else RUN(T, false, false); }                                                     \
+    } while (0)
+    if (dtype == DT_F32) RUN_AS(float);
+    else RUN_AS(bf16);
+#undef RUN_AS
 #undef RUN
     return check_launch("expert_combine_kernel");
 }
 
-extern "C" int mllm_hybrid_route(const void* x, long ld_x, const void* router, const float* router_bias, const void* shared_gate,
-                                 int shared_plain, int softmax_of_chosen, int width, int n_experts, int top, int* choice,
-                                 float* in_weight, float* out_weight, int n_tokens, int dtype, void* stream) {
+extern "C" int mllm_hybrid_route(const void* x, long ld_x, const void* router, const float* router_bias, const float* correction,
+                                 const void* shared_gate, int shared_plain, int rule, float scale, int width, int n_outputs,
+                                 int n_identity, int top, int* choice, float* in_weight, float* out_weight,
+                                 float* identity_weight, int n_tokens, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (top <= 0 || top > n_experts) return fail("route: every token takes between one and all experts");
+    if (top <= 0 || top > n_outputs) return fail("route: every token takes between one and all experts");
     if (shared_plain && shared_gate != nullptr) return fail("route: the shared expert has a gate or none");
+    if (rule < ROUTE_SIGMOID_ON_INPUT || rule > ROUTE_SOFTMAX_OF_ALL) return fail("route: unknown rule");
+    if (n_identity < 0 || n_identity > n_outputs) return fail("route: more identity experts than experts");
+    if (n_identity > 0 && (identity_weight == nullptr || rule == ROUTE_SIGMOID_ON_INPUT))
+        return fail("route: identity experts need weights on the outputs and room for the token's sum of them");
     cudaStream_t s = (cudaStream_t)stream;
     const int pairs = top + (shared_gate != nullptr || shared_plain ? 1 : 0);
-    const size_t shared = sizeof(float) * ((size_t)width + n_experts + 1);
+    const size_t shared = sizeof(float) * ((size_t)width + 2 * (size_t)n_outputs + 1);
     if (shared > 48 * 1024) return fail("route: the token and the scores do not fit shared memory");
-    if (dtype == DT_F32)
-        launch_kernel(g_dependent_launch != 0, route_kernel<float>, dim3(n_tokens), dim3(128), shared, s, (const float*)x, ld_x,
-                      (const float*)router, router_bias, (const float*)shared_gate, shared_plain, softmax_of_chosen, width,
-                      n_experts, top, pairs, choice, in_weight, out_weight);
-    else if (dtype == DT_BF16)
-        launch_kernel(g_dependent_launch != 0, route_kernel<bf16>, dim3(n_tokens), dim3(128), shared, s, (const bf16*)x, ld_x,
-                      (const bf16*)router, router_bias, (const bf16*)shared_gate, shared_plain, softmax_of_chosen, width,
-                      n_experts, top, pairs, choice, in_weight, out_weight);
-    else
-        return fail("route: unknown dtype");
+#define RUN(T)                                                                                                                  \
+    launch_kernel(g_dependent_launch != 0, route_kernel<T>, dim3(n_tokens), dim3(128), shared, s, (const T*)x, ld_x,            \
+                  (const T*)router, router_bias, correction, (const T*)shared_gate, shared_plain, rule, scale, width, n_outputs, \
+                  n_identity, top, pairs, choice, in_weight, out_weight, identity_weight)
+    if (dtype == DT_F32) RUN(float);
+    else if (dtype == DT_BF16) RUN(bf16);
+    else return fail("route: unknown dtype");
+#undef RUN
     return check_launch("route_kernel");
 }
 
+// (gate_of null: experts without a gate matrix, act = the square of relu; identity_weight: see expert_down)
 extern "C" int mllm_hybrid_experts(float* hidden, long ld_hidden, void* act, long ld_act, const void* x, long ld_x,
                                    const int* choice, const float* in_weight, const float* out_weight,
                                    const long long* gate_of, const long long* up_of, const long long* down_of,
-                                   const int* inner_of, long ld_down, int max_inner, int width, int pairs, int n_tokens,
-                                   int assign, int dtype, void* stream) {
+                                   const int* inner_of, long ld_down, int max_inner, int width, int pairs,
+                                   const float* identity_weight, int n_tokens, int assign, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     const size_t shared = sizeof(float) * (size_t)width;
@@ -1463,19 +1575,22 @@ extern "C" int mllm_hybrid_experts(float* hidden, long ld_hidden, void* act, lon
     int down_y = (width + 7) / 8;
     if (down_y > 16) down_y = 16;
     dim3 down_grid(n_tokens, down_y);
-    if (dtype == DT_F32) {
-        launch_kernel(g_dependent_launch != 0, expert_up_kernel<float>, up_grid, dim3(256), shared, s, (float*)act, ld_act,
-                      (const float*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);
-        launch_kernel(g_dependent_launch != 0, expert_down_kernel<float>, down_grid, dim3(256), 0, s, hidden, ld_hidden,
-                      (const float*)act, ld_act, choice, out_weight, down_of, inner_of, ld_down, width, pairs, assign);
-    } else if (dtype == DT_BF16) {
-        launch_kernel(g_dependent_launch != 0, expert_up_kernel<bf16>, up_grid, dim3(256), shared, s, (bf16*)act, ld_act,
-                      (const bf16*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);
-        launch_kernel(g_dependent_launch != 0, expert_down_kernel<bf16>, down_grid, dim3(256), 0, s, hidden, ld_hidden,
-                      (const bf16*)act, ld_act, choice, out_weight, down_of, inner_of, ld_down, width, pairs, assign);
-    } else {
-        return fail("experts: unknown dtype");
-    }
+#define RUN(T)                                                                                                                  \
+    do {                                                                                                                        \
+        if (gate_of != nullptr)                                                                                                 \
+            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, true>, up_grid, dim3(256), shared, s, (T*)act, ld_act,   \
+                          (const T*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);                        \
+        else                                                                                                                    \
+            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, false>, up_grid, dim3(256), shared, s, (T*)act, ld_act,  \
+                          (const T*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);                        \
+        launch_kernel(g_dependent_launch != 0, expert_down_kernel<T>, down_grid, dim3(256), 0, s, hidden, ld_hidden,            \
+                      (const T*)act, ld_act, choice, out_weight, down_of, inner_of, ld_down, width, pairs, assign, (const T*)x, \
+                      ld_x, identity_weight);                                                                                   \
+    } while (0)
+    if (dtype == DT_F32) RUN(float);
+    else if (dtype == DT_BF16) RUN(bf16);
+    else return fail("experts: unknown dtype");
+#undef RUN
     return check_launch("expert kernels");
 }
 

@@ -17,12 +17,12 @@
 MLLM_DEFINE_ERROR_API(mllm_plain)
 
 // ---------------------------------------------------------------------------
-// Embedding: out[t, :] = table[id[t], :] (+ position_table[pos[t], :])
+// Embedding: out[t, :] = scale * table[id[t], :] (+ position_table[pos[t], :])
 // ---------------------------------------------------------------------------
 template <typename W>
 __global__ void embed_kernel(float* __restrict__ out, const int* __restrict__ ids,
                              const int* __restrict__ positions, const W* __restrict__ table,
-                             const W* __restrict__ position_table, int width) {
+                             const W* __restrict__ position_table, int width, float scale) {
     dependents_may_start();
     wait_for_earlier_kernels();
     int t = blockIdx.x;
@@ -30,10 +30,10 @@ __global__ void embed_kernel(float* __restrict__ out, const int* __restrict__ id
     if (position_table != nullptr) {
         long prow = (long)positions[t] * width;
         for (int d = threadIdx.x; d < width; d += blockDim.x)
-            out[(long)t * width + d] = to_f32(table[row + d]) + to_f32(position_table[prow + d]);
+            out[(long)t * width + d] = to_f32(table[row + d]) * scale + to_f32(position_table[prow + d]);
     } else {
         for (int d = threadIdx.x; d < width; d += blockDim.x)
-            out[(long)t * width + d] = to_f32(table[row + d]);
+            out[(long)t * width + d] = to_f32(table[row + d]) * scale;
     }
 }
 
@@ -48,17 +48,17 @@ __global__ void add_rows_kernel(float* __restrict__ hidden, const int* __restric
 }
 
 extern "C" int mllm_plain_embed(float* out, const int* ids, const int* positions, const void* table,
-                                const void* position_table, int n_tokens, int width, int table_dtype,
+                                const void* position_table, int n_tokens, int width, float scale, int table_dtype,
                                 void* stream) {
     if (n_tokens <= 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     int threads = width >= 256 ? 256 : 64;
     if (table_dtype == DT_F32)
         launch_kernel(g_dependent_launch != 0, embed_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, out, ids, positions,
-                      (const float*)table, (const float*)position_table, width);
+                      (const float*)table, (const float*)position_table, width, scale);
     else if (table_dtype == DT_BF16)
         launch_kernel(g_dependent_launch != 0, embed_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, out, ids, positions,
-                      (const bf16*)table, (const bf16*)position_table, width);
+                      (const bf16*)table, (const bf16*)position_table, width, scale);
     else
         return fail("embed: unknown table dtype");
     return check_launch("embed_kernel");

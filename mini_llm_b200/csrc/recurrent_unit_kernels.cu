@@ -3,7 +3,8 @@
 //   norm_rotary_store  a step's projected queries and keys (32-bit) over their root mean square, times a
 //                      gain (over the whole projection, or per head with one gain for all heads), then
 //                      rotary positions on the first rot_dims entries of every head (pairs that are
-//                      neighbours, or half the rotated entries apart); queries go out in the activations'
+//                      neighbours, or half the rotated entries apart), optionally behind a short causal
+//                      convolution over time on every column; queries go out in the activations'
 //                      type, the keys and the values into their cache pages
 //   gated_recurrence   S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t per channel, a_t = exp(-c r_t softplus(lam)),
 //                      r_t and i_t the sigmoids of two gates; the output is S_t times gelu(y_t); state and
@@ -27,7 +28,11 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + l
 // root mean square of the whole projection, gains of that size; 2: every head over its own, one gain of
 // `dim` entries for all heads; 0: none.  layout 0: entries 2i and 2i+1 turn together; 1: entries i and
 // i + rot_dims/2.  Pair i turns by position * inv_freq[i] (the angle in 64-bit, rounded once).  With
-// writes == 0 only the queries are made (the keys and values are another layer's).
+// writes == 0 only the queries are made (the keys and values are another layer's).  With `tap_weights`
+// [columns, taps] every column first passes a short causal convolution, y_t = sum_j w[c, j] u_(t - taps + 1 + j): what
+// lies before this step's portion comes from the request's `tap_state` (the last taps - 1 projected rows, oldest
+// first, 32-bit), which a step of single tokens (tap_moves) also moves on here, each column by the one thread that
+// reads it; after other steps a pass of its own does (another block may still need the rows).
 // One block per token; the token's q and k lie in shared memory in 32-bit.
 // ---------------------------------------------------------------------------
 template <typename T>
@@ -37,7 +42,9 @@ norm_rotary_store_kernel(const float* __restrict__ qkv, long ld, int k_off, int 
                          const float* __restrict__ k_gain, int norm_mode, float eps, int rot_dims, int layout,
                          const double* __restrict__ inv_freq, const int* __restrict__ positions,
                          const int* __restrict__ token_item, const int* __restrict__ block_table, int max_blocks,
-                         int page_size, T* __restrict__ k_pages, T* __restrict__ v_pages, int writes) {
+                         int page_size, T* __restrict__ k_pages, T* __restrict__ v_pages, int writes,
+                         const float* __restrict__ tap_weights, int taps, float* tap_state, long tap_stride, int tap_width,
+                         const int* __restrict__ item_slot, const int* __restrict__ item_start, int tap_moves) {
     dependents_may_start();
     wait_for_earlier_kernels();
     extern __shared__ float shared[];
@@ -50,6 +57,25 @@ norm_rotary_store_kernel(const float* __restrict__ qkv, long ld, int k_off, int 
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
     const int p = positions[t];
     const float* row = qkv + (long)t * ld;
+    const int item = token_item[t];
+    const int local = taps > 1 ? p - item_start[item] : 0;          // tokens of this request before t in this step
+    float* held = taps > 1 ? tap_state + (long)item_slot[item] * tap_stride : nullptr;
+    auto column = [&](int c) {
+        const float mine = row[c];
+        if (taps <= 0) return mine;
+        const float* w = tap_weights + (long)c * taps;
+        float acc = 0.0f;
+        for (int back = taps - 1; back >= 1; back--) {
+            const float v = local >= back ? row[c - (long)back * ld] : held[(long)(taps - 1 + local - back) * tap_width + c];
+            acc = fmaf(w[taps - 1 - back], v, acc);
+        }
+        acc = fmaf(w[taps - 1], mine, acc);
+        if (tap_moves && taps > 1) {
+            for (int s = 0; s + 1 < taps - 1; s++) held[(long)s * tap_width + c] = held[(long)(s + 1) * tap_width + c];
+            held[(long)(taps - 2) * tap_width + c] = mine;
+        }
+        return acc;
+    };
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         double s, c;
         sincos((double)p * inv_freq[i], &s, &c);
@@ -57,14 +83,14 @@ norm_rotary_store_kernel(const float* __restrict__ qkv, long ld, int k_off, int 
         turn[2 * i + 1] = (float)s;
     }
     const int q_width = heads * dim, k_width = kv_heads * dim;
-    for (int c = threadIdx.x; c < q_width; c += blockDim.x) x[c] = row[c];
+    for (int c = threadIdx.x; c < q_width; c += blockDim.x) x[c] = column(c);
     long slot = 0;
     if (writes) {
-        slot = (long)block_table[(long)token_item[t] * max_blocks + p / page_size] * page_size + (p % page_size);
-        for (int c = threadIdx.x; c < k_width; c += blockDim.x) x[q_width + c] = row[k_off + c];
-        // the values leave first: they may be the keys as projected
+        slot = (long)block_table[(long)item * max_blocks + p / page_size] * page_size + (p % page_size);
+        for (int c = threadIdx.x; c < k_width; c += blockDim.x) x[q_width + c] = column(k_off + c);
+        // the values leave first: they may be the keys as projected (then the thread that filtered a column has it)
         for (int c = threadIdx.x; c < kv_heads * vdim; c += blockDim.x)
-            v_pages[slot * kv_heads * vdim + c] = from_f32<T>(row[v_off + c]);
+            v_pages[slot * kv_heads * vdim + c] = from_f32<T>(v_off == k_off ? x[q_width + c] : column(v_off + c));
     }
     __syncthreads();
     if (norm_mode == 1) {
@@ -116,11 +142,17 @@ extern "C" int mllm_unit_norm_rotary_store(const float* qkv, long ld, int k_off,
                                            int norm_mode, float eps, int rot_dims, int layout, const double* inv_freq,
                                            const int* positions, const int* token_item, const int* block_table,
                                            int max_blocks, int page_size, void* k_pages, void* v_pages, int writes,
+                                           const float* tap_weights, int taps, float* tap_state, long tap_stride,
+                                           int tap_width, const int* item_slot, const int* item_start, int tap_moves,
                                            int n_tokens, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     if (heads <= 0 || dim <= 0 || (writes && (kv_heads <= 0 || vdim <= 0))) return fail("norm_rotary_store: sizes must be positive");
     if (rot_dims < 0 || rot_dims % 2 != 0 || rot_dims > dim) return fail("norm_rotary_store: an even number of at most dim entries is rotated");
     if (norm_mode < 0 || norm_mode > 2 || layout < 0 || layout > 1) return fail("norm_rotary_store: unknown norm or layout");
+    if (tap_weights == nullptr) taps = 0;
+    if (taps < 0 || (taps > 1 && (tap_state == nullptr || item_slot == nullptr || item_start == nullptr)))
+        return fail("norm_rotary_store: taps need the requests' last rows");
+    if (writes && v_off == k_off && vdim != dim) return fail("norm_rotary_store: values that are the keys have their size");
     cudaStream_t s = (cudaStream_t)stream;
     const int all_heads = heads + (writes ? kv_heads : 0);
     const size_t shared = sizeof(float) * ((size_t)rot_dims + 2 + all_heads + 33 + (size_t)all_heads * dim);
@@ -132,7 +164,8 @@ extern "C" int mllm_unit_norm_rotary_store(const float* qkv, long ld, int k_off,
             return fail("norm_rotary_store: the shared memory was refused");                                                     \
         launch_kernel(g_dependent_launch != 0, norm_rotary_store_kernel<T>, dim3(n_tokens), dim3(256), shared, s, qkv, ld, k_off, \
                       v_off, heads, kv_heads, dim, vdim, (T*)q_out, ld_q, q_gain, k_gain, norm_mode, eps, rot_dims, layout,      \
-                      inv_freq, positions, token_item, block_table, max_blocks, page_size, (T*)k_pages, (T*)v_pages, writes);    \
+                      inv_freq, positions, token_item, block_table, max_blocks, page_size, (T*)k_pages, (T*)v_pages, writes,     \
+                      tap_weights, taps, tap_state, tap_stride, tap_width, item_slot, item_start, tap_moves);                    \
     } while (0)
     if (dtype == DT_F32) RUN(float);
     else if (dtype == DT_BF16) RUN(bf16);

@@ -225,6 +225,16 @@ extern "C" int mllm_sequence_norm_taps_step(void* out, const float* x, const flo
     return check_launch("norm_taps_step_kernel");
 }
 
+// The move of the state alone, after a kernel that filtered 32-bit rows itself.
+extern "C" int mllm_sequence_taps_state(float* state, long state_stride, const float* h, long ld_h, const int* item_slot,
+                                        const int* item_offset, const int* item_count, int n_items, int width, int taps,
+                                        void* stream) {
+    if (n_items <= 0 || taps <= 1) return 0;
+    launch_kernel(g_dependent_launch != 0, causal_taps_state_kernel<float>, dim3(n_items), dim3(width >= 256 ? 256 : 64), 0,
+                  (cudaStream_t)stream, state, state_stride, h, ld_h, item_slot, item_offset, item_count, width, taps);
+    return check_launch("causal_taps_state_kernel");
+}
+
 // (Not in place: the state's move reads the step's inputs after the filter has run.)
 extern "C" int mllm_sequence_causal_taps(void* out, long ld_out, const void* h, long ld_h, const float* w, const float* bias,
                                          float* state, long state_stride, const int* positions, const int* token_item,

@@ -77,9 +77,9 @@ class Kernels:
         self.launches += 1
         return ops.resolve_tokens(token_ids, kept)
 
-    def embed(self, out, token_ids, positions, table, position_table=None):
+    def embed(self, out, token_ids, positions, table, position_table=None, scale=1.0):
         self.launches += 1
-        return ops.embed(out, token_ids, positions, table, position_table)
+        return ops.embed(out, token_ids, positions, table, position_table, scale)
 
     def add_position_rows(self, hidden, positions, table):
         self.launches += 1
@@ -124,31 +124,34 @@ class Kernels:
                                    cache.block_table, cache.page_size, cache.k_pages, cache.v_pages, cache.writes)
 
     def capped_attention(self, ctx, out, q, cache, n_heads, n_kv_heads, dim, vdim, scale, cap=0.0, window=0, chunk=0,
-                         gate=None, sink=None):
+                         gate=None, sink=None, keep=0):
         """Attention whose weights stay 32-bit, with a cap on the scores and values of a size of
-        their own; the mask is causal, over the last ``window`` positions or within blocks of
-        ``chunk`` positions; ``gate`` [T, heads] opens each head's result by its sigmoid; ``sink`` [heads] adds
+        their own; the mask is causal, over the last ``window`` positions (and the first ``keep``) or within
+        blocks of ``chunk`` positions; ``gate`` [T, heads] opens each head's result by its sigmoid; ``sink`` [heads] adds
         exp(sink[h]) to head h's denominator.  Steps with
         prompt portions take the tiles (tokens of a request side by side share the cached rows they
         read); steps of single tokens, and sizes the tiles do not take, one block per (token, head)."""
         self.launches += 1
         n = q.shape[0]
-        if (not self.plain_only and ctx.decode_only and n <= SPLIT_ATTENTION_MAX_ROWS and dim == vdim
-                and dim in ops.SPLIT_ATTENTION_HEAD_SIZES and q.dtype == torch.bfloat16 and q.stride(0) % 8 == 0):
+        row = ops.split_attention_row(dim, vdim)
+        if (not self.plain_only and ctx.decode_only and n <= SPLIT_ATTENTION_MAX_ROWS and row is not None
+                and q.dtype == torch.bfloat16 and q.stride(0) % 8 == 0):
             # single tokens: each token's keys in chunks over many CTAs, merged by the last to arrive
             # (its exponentials, weights and sums are 32-bit, which this attention asks for)
             pairs = n * n_heads
             span = 64 if pairs < 64 else (128 if pairs < 128 else (256 if pairs < 256 else 512))
             reach = cache.block_table.shape[1] * cache.page_size
-            acc, ml, counters = self._scratch(ctx, SPLIT_ATTENTION_MAX_ROWS * n_heads, -(-reach // 64), dim)
+            if window:
+                reach = min(reach, window + keep)              # the most keys a token sees
+            acc, ml, counters = self._scratch(ctx, SPLIT_ATTENTION_MAX_ROWS * n_heads, -(-reach // 64), row)
             self.chose("capped_attention", "split_attention", n, n_heads, dim, vdim)
             return ops.split_attention(out, q, cache.k_pages, cache.v_pages, cache.block_table, ctx.positions, ctx.token_item,
                                        n_heads, n_kv_heads, dim, cache.page_size, scale, window, span, -(-reach // span), acc,
-                                       ml, counters, cap=cap, block=chunk, gate=gate, sink=sink)
+                                       ml, counters, cap=cap, block=chunk, gate=gate, sink=sink, value_size=vdim, keep=keep)
         tiled = not ctx.decode_only and ops.capped_attention_tiled_takes(dim, vdim, q.dtype)
         self.chose("capped_attention", "capped_attention_tiled" if tiled else "capped_attention_plain", q.shape[0], n_heads, dim, vdim)
         return ops.capped_attention(out, q, cache.k_pages, cache.v_pages, cache.block_table, ctx.positions, ctx.token_item,
-                                    n_heads, n_kv_heads, dim, vdim, cache.page_size, scale, cap, window, tiled, chunk, gate, sink)
+                                    n_heads, n_kv_heads, dim, vdim, cache.page_size, scale, cap, window, tiled, chunk, gate, sink, keep)
 
     def linear_recurrence(self, ctx, out, q, k, v, gate_a, gate_b, log_rate, step_bias, state, heads, qk_heads, dim, vdim,
                           delta, unit_norm=False, q_scale=1.0, skip=None, writes=True, channel_decay=False):
@@ -157,16 +160,15 @@ class Kernels:
                                      ctx.item_count, heads, qk_heads, dim, vdim, delta, unit_norm, q_scale, skip, writes,
                                      channel_decay)
 
-    def route(self, x, router, shared_gate, top, choice, in_weight, out_weight, bias=None, softmax_of_chosen=False,
-              shared_plain=False):
+    def route(self, x, router, shared_gate, top, choice, in_weight, out_weight, **how):
         self.launches += 1
-        return ops.route(x, router, shared_gate, top, choice, in_weight, out_weight, bias, softmax_of_chosen, shared_plain)
+        return ops.route(x, router, shared_gate, top, choice, in_weight, out_weight, **how)
 
     def experts(self, hidden, act, x, choice, in_weight, out_weight, gate_of, up_of, down_of, inner_of, max_inner, pairs,
-                ld_down=None, assign=False):
+                ld_down=None, assign=False, identity_weight=None):
         self.launches += 2
         return ops.experts(hidden, act, x, choice, in_weight, out_weight, gate_of, up_of, down_of, inner_of, max_inner, pairs,
-                           ld_down, assign)
+                           ld_down, assign, identity_weight)
 
     EXPERTS_AT_ONCE_TOKENS = 32    # from here on a step's tokens go through all experts as two products
 
@@ -177,18 +179,25 @@ class Kernels:
         return (not self.plain_only and n_tokens >= self.EXPERTS_AT_ONCE_TOKENS and isinstance(x, torch.Tensor)
                 and ops.gemm_takes(x, up_matrix) and down_matrix.shape[1] % 8 == 0 and down_matrix.shape[0] >= 16)
 
-    def expert_combine(self, act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs):
+    def expert_combine(self, act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs, **more):
         self.launches += 1
-        return ops.expert_combine(act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs)
+        return ops.expert_combine(act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs, **more)
 
     # ---- norms on a sublayer's output, query and key norms with rotary positions, the gated linear recurrence ----
     def norm_rotary_store(self, ctx, cache, qkv, q_out, k_off, v_off, heads, kv_heads, dim, vdim, q_gain, k_gain, norm, eps,
-                          rot_dims, layout, inv_freq):
+                          rot_dims, layout, inv_freq, taps=None):
+        """``taps``: (weights, state): a short convolution over every projected column goes first, in the same kernel
+        (and moves its state there in a step of single tokens, else in a pass of its own)."""
         self.launches += 1
         writes = bool(cache.writes)
+        if taps is not None:
+            single = bool(ctx.decode_only)
+            self.launches += 0 if single or taps[0].shape[1] == 1 else 1
+            taps = (*taps, ctx.item_slot, ctx.item_start, ctx.item_offset, ctx.item_count, single)
         return ops.norm_rotary_store(qkv, k_off, v_off, heads, kv_heads, dim, vdim, q_out, q_gain, k_gain, norm, eps, rot_dims,
                                      layout, inv_freq, ctx.positions, ctx.token_item, cache.block_table if writes else None,
-                                     cache.page_size, cache.k_pages if writes else None, cache.v_pages if writes else None, writes)
+                                     cache.page_size, cache.k_pages if writes else None, cache.v_pages if writes else None, writes,
+                                     taps)
 
     def gated_recurrence(self, ctx, out, u, y, gates, bias_r, bias_i, lam, decay_scale, state, block_width, writes=True):
         self.launches += 1

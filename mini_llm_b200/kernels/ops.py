@@ -68,7 +68,7 @@ def _ptr(t):
     return None if t is None else t.data_ptr()
 
 
-_embed = Function("plain", "mllm_plain_embed", [P, P, P, P, P, I, I, I, P])
+_embed = Function("plain", "mllm_plain_embed", [P, P, P, P, P, I, I, F, I, P])
 _add_rows = Function("plain", "mllm_plain_add_rows", [P, P, P, I, I, I, P])
 _layernorm = Function("plain", "mllm_plain_layernorm", [P, P, P, P, P, I, I, F, I, P])
 _linear = Function("plain", "mllm_plain_linear", [P, P, P, P, I, I, I, L, L, I, I, I, P])
@@ -78,8 +78,8 @@ _attention = Function("plain", "mllm_plain_attention",
 _sample_rows = Function("sampling", "mllm_sampling_sample_rows", [P, P, L, I, I, P, P, P, P, P])
 
 
-def embed(out, token_ids, positions, table, position_table=None):
-    """out[t] = table[token_ids[t]] (+ position_table[positions[t]]); out is fp32 [T, width]."""
+def embed(out, token_ids, positions, table, position_table=None, scale=1.0):
+    """out[t] = scale * table[token_ids[t]] (+ position_table[positions[t]]); out is fp32 [T, width]."""
     _check(out, "embed.out", torch.float32, 2)
     _check(token_ids, "embed.token_ids", torch.int32, 1)
     _check(table, "embed.table", None, 2)
@@ -94,7 +94,7 @@ def embed(out, token_ids, positions, table, position_table=None):
         if position_table.shape[1] != width or not position_table.is_contiguous():
             raise KernelError("embed: position table has another width")
     _embed(out.data_ptr(), token_ids.data_ptr(), _ptr(positions), table.data_ptr(), _ptr(position_table),
-           n, width, dtype_code(table.dtype), _stream())
+           n, width, float(scale), dtype_code(table.dtype), _stream())
     return out
 
 
@@ -228,11 +228,19 @@ class _SkinnyParams(ctypes.Structure):
 
 
 _skinny = Function("decode", "mllm_decode_skinny_linear", [ctypes.POINTER(_SkinnyParams), P])
-_split_attention = Function("decode", "mllm_decode_split_attention_sink",
-                            [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, F, F, I, I, P, L, P, I, I, P, P, P, P])
+_split_attention = Function("decode", "mllm_decode_split_attention_kept",
+                            [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, F, I, I, I, P, L, P, I, I, P, P, P, P])
 
 SKINNY_MAX_SMEM = 200 * 1024
 SPLIT_ATTENTION_HEAD_SIZES = (16, 32, 64, 128, 256)
+
+
+def split_attention_row(dim, vdim):
+    """Floats of a scratch row for keys of ``dim`` and values of ``vdim`` entries: the least of the head sizes that
+    holds both, or None where split_attention does not take them (other sizes than multiples of 8 up to 256)."""
+    if dim <= 0 or vdim <= 0 or dim % 8 != 0 or vdim % 8 != 0:
+        return None
+    return next((size for size in SPLIT_ATTENTION_HEAD_SIZES if size >= max(dim, vdim)), None)
 
 
 def skinny_linear_takes(m, k) -> bool:
@@ -303,14 +311,17 @@ def skinny_linear(out, x, w, bias=None, epilogue="store", norm=None, scatter=Non
 
 
 def split_attention(out, q, k_pages, v_pages, block_table, positions, token_item, n_heads, n_kv_heads, head_size,
-                    page_size, scale, window, chunk, max_chunks, part_acc, part_ml, counters, cap=0.0, block=0, gate=None, sink=None):
+                    page_size, scale, window, chunk, max_chunks, part_acc, part_ml, counters, cap=0.0, block=0, gate=None, sink=None,
+                    value_size=None, keep=0):
     """Causal attention over the paged cache for few tokens: one CTA per (token, head, chunk
     of ``chunk`` keys); needs fp32 scratch ``part_acc`` [T*H*max_chunks*D], ``part_ml``
     [T*H*max_chunks*2] and zeroed int32 ``counters`` [T*H] (left zero).  ``cap`` > 0: the scores
     are capped, cap * tanh(score / cap).  ``block`` > 0: a query sees only the keys of its own block of
     ``block`` positions (blocks counted from position 0).  ``gate`` fp32 [T, >= heads]: head h's result
     is multiplied by sigmoid(gate[t, h]).  ``sink`` fp32 [heads]: exp(sink[h]) joins head h's denominator.
-    Scores, weights and sums are 32-bit."""
+    ``value_size``: entries of a value where they are not ``head_size`` (then both are multiples of 8 up to 256 and the
+    scratch is sized for ``split_attention_row``).  ``keep``: the first ``keep`` keys stay visible behind the window.
+    ``max_chunks`` chunks must cover the most keys a token may see.  Scores, weights and sums are 32-bit."""
     _check(out, "split_attention.out", torch.bfloat16, 2)
     _check(q, "split_attention.q", torch.bfloat16, 2)
     _check(k_pages, "split_attention.k_pages", torch.bfloat16)
@@ -321,14 +332,19 @@ def split_attention(out, q, k_pages, v_pages, block_table, positions, token_item
     _check(counters, "split_attention.counters", torch.int32)
     n = q.shape[0]
     cells = n * n_heads * max_chunks
-    if head_size not in SPLIT_ATTENTION_HEAD_SIZES:
-        raise KernelError(f"split_attention does not take head size {head_size}")
-    if q.shape[1] != n_heads * head_size or out.shape != q.shape:
+    vdim = head_size if value_size is None else int(value_size)
+    row = split_attention_row(head_size, vdim)
+    if row is None or (value_size is None and row != head_size):
+        raise KernelError(f"split_attention does not take head size {head_size}" + (f" with values of {vdim}" if value_size is not None else ""))
+    if q.shape[1] != n_heads * head_size or out.shape != (n, n_heads * vdim):
         raise KernelError("split_attention: q / out do not have heads * head_size columns")
-    if part_acc.numel() < cells * head_size or part_ml.numel() < cells * 2 or counters.numel() < n * n_heads:
+    if part_acc.numel() < cells * row or part_ml.numel() < cells * 2 or counters.numel() < n * n_heads:
         raise KernelError("split_attention: scratch too small")
-    if max_chunks * chunk < page_size * block_table.shape[1]:
-        raise KernelError("split_attention: the chunks do not cover the longest block table")
+    reach = page_size * block_table.shape[1]
+    if max_chunks * chunk < (min(reach, window + keep) if window else reach):
+        raise KernelError("split_attention: the chunks do not cover the longest block table (or the window)")
+    if keep < 0 or (keep and block):
+        raise KernelError("split_attention: kept first keys go with a window, not with blocks of positions")
     if gate is not None:
         _check(gate, "split_attention.gate", torch.float32, 2)
         if gate.shape[0] < n or gate.shape[1] < n_heads or gate.stride(1) != 1:
@@ -336,8 +352,8 @@ def split_attention(out, q, k_pages, v_pages, block_table, positions, token_item
     _check_sink(sink, n_heads, "split_attention")
     _split_attention(out.data_ptr(), out.stride(0), q.data_ptr(), q.stride(0), k_pages.data_ptr(), v_pages.data_ptr(),
                      block_table.data_ptr(), block_table.shape[1], positions.data_ptr(), token_item.data_ptr(), n,
-                     n_heads, n_kv_heads, head_size, page_size, float(scale), float(cap or 0.0), int(window or 0), int(block or 0),
-                     _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(sink), int(chunk), int(max_chunks), part_acc.data_ptr(),
+                     n_heads, n_kv_heads, head_size, vdim, page_size, float(scale), float(cap or 0.0), int(window or 0), int(block or 0),
+                     int(keep), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(sink), int(chunk), int(max_chunks), part_acc.data_ptr(),
                      part_ml.data_ptr(), counters.data_ptr(), _stream())
     return out
 
@@ -1201,7 +1217,7 @@ def rotary_store(qkv, k_off, v_off, heads, kv_heads, dim, vdim, rot_dims, inv_fr
 
 
 _capped_attention = Function("hybrid", "mllm_hybrid_capped_attention",
-                             [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, F, I, I, P, L, P, I, I, P])
+                             [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, F, I, I, I, P, L, P, I, I, P])
 
 
 def capped_attention_tiled_takes(dim, vdim, dtype=torch.bfloat16) -> bool:
@@ -1214,11 +1230,11 @@ def capped_attention_tiled_takes(dim, vdim, dtype=torch.bfloat16) -> bool:
 
 
 def capped_attention(out, q, k_pages, v_pages, block_table, positions, token_item, n_heads, n_kv_heads, dim, vdim,
-                     page_size, scale, cap=0.0, window=0, tiled=False, chunk=0, gate=None, sink=None):
+                     page_size, scale, cap=0.0, window=0, tiled=False, chunk=0, gate=None, sink=None, keep=0):
     """Causal attention of every token of the step over its request's pages, keys of ``dim`` and
     values of ``vdim`` entries per head, score = cap * tanh(q . k * scale / cap) (``cap`` 0: no cap);
-    scores, weights and the weighted sum in 32-bit.  ``window`` > 0: the last ``window`` positions only;
-    ``chunk`` > 0: only keys of the query's own block of ``chunk`` positions (blocks counted from
+    scores, weights and the weighted sum in 32-bit.  ``window`` > 0: the last ``window`` positions only, and the
+    first ``keep`` of the sequence; ``chunk`` > 0: only keys of the query's own block of ``chunk`` positions (blocks counted from
     position 0).  ``gate`` fp32 [T, >= heads]: head h's result is multiplied by sigmoid(gate[t, h]).
     ``sink`` fp32 [heads]: the softmax's denominator also holds exp(sink[h]), a term with no key and no value.
     ``tiled``: consecutive tokens of a request share the cached rows they read (for steps with prompt
@@ -1238,10 +1254,12 @@ def capped_attention(out, q, k_pages, v_pages, block_table, positions, token_ite
         if gate.shape[0] < n or gate.shape[1] < n_heads or gate.stride(1) != 1:
             raise KernelError("capped_attention: one gate per token and head")
     _check_sink(sink, n_heads, "capped_attention")
+    if keep < 0 or (keep and chunk):
+        raise KernelError("capped_attention: kept first keys go with a window, not with blocks of positions")
     _capped_attention(out.data_ptr(), out.stride(0), q.data_ptr(), q.stride(0), k_pages.data_ptr(), v_pages.data_ptr(),
                       block_table.data_ptr(), block_table.shape[1], positions.data_ptr(), token_item.data_ptr(), n, n_heads,
                       n_kv_heads, dim, vdim, page_size, float(scale), float(cap or 0.0), int(window or 0), int(chunk or 0),
-                      _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(sink), int(bool(tiled)), dtype_code(q.dtype),
+                      int(keep), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(sink), int(bool(tiled)), dtype_code(q.dtype),
                       _stream())
     return out
 
@@ -1326,18 +1344,27 @@ def linear_recurrence(out, q, k, v, gate_a, gate_b, log_rate, step_bias, state, 
     return out
 
 
-_route = Function("hybrid", "mllm_hybrid_route", [P, L, P, P, P, I, I, I, I, I, P, P, P, I, I, P])
-_experts = Function("hybrid", "mllm_hybrid_experts", [P, L, P, L, P, L, P, P, P, P, P, P, P, L, I, I, I, I, I, I, P])
-_expert_combine = Function("hybrid", "mllm_hybrid_expert_combine", [P, L, P, L, P, P, P, I, I, I, I, I, I, I, P])
+_route = Function("hybrid", "mllm_hybrid_route", [P, L, P, P, P, P, I, I, F, I, I, I, I, P, P, P, P, I, I, P])
+_experts = Function("hybrid", "mllm_hybrid_experts", [P, L, P, L, P, L, P, P, P, P, P, P, P, L, I, I, I, P, I, I, I, P])
+_expert_combine = Function("hybrid", "mllm_hybrid_expert_combine",
+                           [P, L, P, L, P, P, P, I, I, I, I, I, I, P, L, P, L, P, I, I, I, I, P])
+ROUTE_RULES = {"sigmoid_on_input": 0, "softmax_of_chosen": 1, "softmax_of_all": 2}
 
 
-def route(x, router, shared_gate, top, choice, in_weight, out_weight, bias=None, softmax_of_chosen=False, shared_plain=False):
-    """Per row of ``x``: sigmoid scores of ``router`` [experts, width] (sums in 32-bit), the ``top``
-    largest with their scores as input weights; with ``shared_gate`` [1, width] one more pair per
-    token: expert ``experts``, input weight 1, output weight sigmoid(shared_gate . x); ``shared_plain``:
-    that pair with output weight 1 and no gate.  ``softmax_of_chosen``: the logits (plus ``bias`` fp32
-    [experts]) rank the experts, and the chosen ones get input weight 1 and, as output weight, the
-    softmax over the chosen logits only.  choice int32, in_weight / out_weight fp32: [T * pairs]."""
+def route(x, router, shared_gate, top, choice, in_weight, out_weight, bias=None, rule="sigmoid_on_input", shared_plain=False,
+          correction=None, n_identity=0, scale=1.0, identity_weight=None):
+    """Per row of ``x``: the outputs of ``router`` [outputs, width] (sums in 32-bit, plus ``bias`` fp32 [outputs]), of which the
+    ``top`` largest are chosen (the lower index wins a tie).  ``rule``:
+    "sigmoid_on_input": sigmoid scores rank them and weigh the chosen experts' inputs;
+    "softmax_of_chosen": the logits rank them; the chosen ones get input weight 1 and, as output weight, the softmax over
+    the chosen logits only;
+    "softmax_of_all": s = the softmax over all outputs; s + ``correction`` (fp32 [outputs]) ranks them; output weights
+    s / (sum of the chosen s + 1e-20) * ``scale``.
+    The last ``n_identity`` outputs are identity experts (the output is the token itself): such a choice is stored as
+    -1 with weight 0, and the token's weights of that kind are summed in ``identity_weight`` fp32 [T].
+    With ``shared_gate`` [1, width] one more pair per token: expert ``outputs - n_identity``, input weight 1, output weight
+    sigmoid(shared_gate . x); ``shared_plain``: that pair with output weight 1 and no gate.  choice int32, in_weight /
+    out_weight fp32: [T * pairs]."""
     _check(x, "route.x", None, 2)
     _check(router, "route.router", x.dtype, 2)
     _check(choice, "route.choice", torch.int32, 1)
@@ -1347,55 +1374,87 @@ def route(x, router, shared_gate, top, choice, in_weight, out_weight, bias=None,
     pairs = top + (1 if shared_gate is not None or shared_plain else 0)
     if router.shape[1] != width or not router.is_contiguous() or min(choice.shape[0], in_weight.shape[0], out_weight.shape[0]) < n * pairs:
         raise KernelError("route: sizes do not agree")
-    if bias is not None:
-        _check(bias, "route.bias", torch.float32, 1)
-        if bias.shape[0] != router.shape[0]:
-            raise KernelError("route: one bias per expert")
+    for name, t in (("bias", bias), ("correction", correction)):
+        if t is not None:
+            _check(t, f"route.{name}", torch.float32, 1)
+            if t.shape[0] != router.shape[0]:
+                raise KernelError(f"route: one {name} per expert")
+    if n_identity and identity_weight is None:
+        raise KernelError("route: identity experts need room for the tokens' weights of them")
+    if identity_weight is not None:
+        _check(identity_weight, "route.identity_weight", torch.float32, 1)
+        if identity_weight.shape[0] < n:
+            raise KernelError("route: one identity weight per token")
     if shared_gate is not None:
         _check(shared_gate, "route.shared_gate", x.dtype)
         if shared_gate.numel() != width or not shared_gate.is_contiguous():
             raise KernelError("route: the shared expert's gate is one row of the width")
-    _route(x.data_ptr(), x.stride(0), router.data_ptr(), _ptr(bias), _ptr(shared_gate), int(bool(shared_plain)),
-           int(bool(softmax_of_chosen)), width, router.shape[0], top, choice.data_ptr(), in_weight.data_ptr(),
-           out_weight.data_ptr(), n, dtype_code(x.dtype), _stream())
+    _route(x.data_ptr(), x.stride(0), router.data_ptr(), _ptr(bias), _ptr(correction), _ptr(shared_gate), int(bool(shared_plain)),
+           ROUTE_RULES[rule], float(scale), width, router.shape[0], int(n_identity), top, choice.data_ptr(), in_weight.data_ptr(),
+           out_weight.data_ptr(), _ptr(identity_weight), n, dtype_code(x.dtype), _stream())
+
+
+def _check_identity(identity_weight, x, n, who):
+    if identity_weight is not None:
+        _check(identity_weight, f"{who}.identity_weight", torch.float32, 1)
+        if identity_weight.shape[0] < n or x is None or x.shape[0] < n:
+            raise KernelError(f"{who}: one identity weight and one row per token")
 
 
 def experts(hidden, act, x, choice, in_weight, out_weight, gate_of, up_of, down_of, inner_of, max_inner, pairs, ld_down=None,
-            assign=False):
+            assign=False, identity_weight=None):
     """hidden[t] += sum over the token's ``pairs`` of out_weight * W_down[e] (silu(W_gate[e] x') * (W_up[e] x')),
     x' = in_weight * x[t] rounded to the activations' type; expert e's matrices are named by the
     int64 pointer tables ``gate_of``, ``up_of``, ``down_of`` and its inner size by ``inner_of`` (int32);
     the rows of every down matrix lie ``ld_down`` elements apart (None: ``max_inner``, for experts of
-    one size that are stored each by itself).  ``act`` [T * pairs, max_inner] is scratch.  ``assign``: ``hidden`` is set
+    one size that are stored each by itself).  ``gate_of`` None: experts without a gate matrix,
+    W_down[e] relu(W_up[e] x')^2.  ``act`` [T * pairs, max_inner] is scratch.  A pair whose choice is negative has no
+    expert; with ``identity_weight`` [T] identity_weight[t] * x[t] joins the sum.  ``assign``: ``hidden`` is set
     to the sum instead of added to."""
     _check(hidden, "experts.hidden", torch.float32, 2)
     _check(x, "experts.x", None, 2)
     _check(act, "experts.act", x.dtype, 2)
     for name, t in (("gate_of", gate_of), ("up_of", up_of), ("down_of", down_of)):
-        _check(t, f"experts.{name}", torch.int64, 1)
+        if t is not None or name != "gate_of":
+            _check(t, f"experts.{name}", torch.int64, 1)
     _check(inner_of, "experts.inner_of", torch.int32, 1)
     n, width = x.shape
     if hidden.shape != (n, width) or act.shape[0] < n * pairs or act.shape[1] < max_inner:
         raise KernelError("experts: sizes do not agree")
+    _check_identity(identity_weight, x, n, "experts")
     _experts(hidden.data_ptr(), hidden.stride(0), act.data_ptr(), act.stride(0), x.data_ptr(), x.stride(0), choice.data_ptr(),
-             in_weight.data_ptr(), out_weight.data_ptr(), gate_of.data_ptr(), up_of.data_ptr(), down_of.data_ptr(),
-             inner_of.data_ptr(), int(ld_down if ld_down is not None else max_inner), int(max_inner), width, int(pairs), n,
-             int(bool(assign)), dtype_code(x.dtype), _stream())
+             in_weight.data_ptr(), out_weight.data_ptr(), _ptr(gate_of), up_of.data_ptr(), down_of.data_ptr(),
+             inner_of.data_ptr(), int(ld_down if ld_down is not None else max_inner), int(max_inner), width, int(pairs),
+             _ptr(identity_weight), n, int(bool(assign)), dtype_code(x.dtype), _stream())
     return hidden
 
 
-def expert_combine(act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs):
+def expert_combine(act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs, gated=True, hidden=None, x=None,
+                   identity_weight=None, assign=False):
     """For the products over all experts at once: ``gu`` [T, 2 * total] holds every expert's gate and
     up results ([gates | ups], routed expert e in columns [e * inner, (e + 1) * inner), the shared
     expert behind them); act[t, c] = silu(s g) * (s u) * out_weight with s the token's input weight
-    for the column's expert, or 0 for an expert it did not choose.  act: [T, total]."""
+    for the column's expert, or 0 for an expert it did not choose.  act: [T, total].  ``gated`` false: ``gu`` [T, total]
+    holds the ups alone and act[t, c] = relu(s u)^2 * out_weight.  With ``identity_weight`` [T] the fp32 ``hidden``
+    [T, width] also gets identity_weight[t] * x[t] (``assign``: is set to it)."""
     _check(act, "expert_combine.act", gu.dtype, 2)
     _check(gu, "expert_combine.gu", None, 2)
     n, total = act.shape
-    if gu.shape != (n, 2 * total) or total < n_experts * inner or (pairs == top and total != n_experts * inner):
+    if gu.shape != (n, (2 if gated else 1) * total) or total < n_experts * inner or (pairs == top and total != n_experts * inner):
         raise KernelError("expert_combine: sizes do not agree")
+    _check_identity(identity_weight, x, n, "expert_combine")
+    width = 0
+    if identity_weight is not None:
+        _check(hidden, "expert_combine.hidden", torch.float32, 2)
+        _check(x, "expert_combine.x", gu.dtype, 2)
+        width = x.shape[1]
+        if hidden.shape != (n, width):
+            raise KernelError("expert_combine: the stream and the tokens have another shape")
     _expert_combine(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.stride(0), choice.data_ptr(), in_weight.data_ptr(),
-                    out_weight.data_ptr(), n_experts, inner, total, top, pairs, n, dtype_code(gu.dtype), _stream())
+                    out_weight.data_ptr(), n_experts, inner, total, top, pairs, int(bool(gated)),
+                    hidden.data_ptr() if width else None, hidden.stride(0) if width else 0, x.data_ptr() if width else None,
+                    x.stride(0) if width else 0, _ptr(identity_weight), width, int(bool(assign)), n, dtype_code(gu.dtype),
+                    _stream())
     return act
 
 
@@ -1483,7 +1542,8 @@ def gated_act(out, gu, activation="silu"):
 # ---- norms on a sublayer's output, query and key norms with rotary positions, gated linear recurrence ----
 
 _norm_rotary_store = Function("unit", "mllm_unit_norm_rotary_store",
-                              [P, L, I, I, I, I, I, I, P, L, P, P, I, F, I, I, P, P, P, P, I, I, P, P, I, I, I, P])
+                              [P, L, I, I, I, I, I, I, P, L, P, P, I, F, I, I, P, P, P, P, I, I, P, P, I, P, I, P, L, I, P, P, I, I, I, P])
+_taps_state = Function("sequence", "mllm_sequence_taps_state", [P, L, P, L, P, P, P, I, I, I, P])
 _gated_recurrence = Function("unit", "mllm_unit_gated_recurrence",
                              [P, L, P, L, P, L, P, L, P, P, P, F, P, L, P, P, P, I, I, I, I, I, I, P])
 _add_normed_cast = Function("unit", "mllm_unit_add_normed_cast", [P, P, P, F, P, I, I, I, P])
@@ -1492,7 +1552,7 @@ QK_NORMS = {None: 0, "none": 0, "whole": 1, "head": 2}
 
 
 def norm_rotary_store(qkv, k_off, v_off, heads, kv_heads, dim, vdim, q_out, q_gain, k_gain, norm, eps, rot_dims, layout, inv_freq,
-                      positions, token_item, block_table, page_size, k_pages, v_pages, writes=True):
+                      positions, token_item, block_table, page_size, k_pages, v_pages, writes=True, taps=None):
     """Rows of the fp32 ``qkv`` hold the projected [q | k | v] (k from column ``k_off``, v from ``v_off``; ``v_off`` may
     equal ``k_off``: the values are then the keys as projected).  ``norm`` "whole": q and k are divided by the root mean
     square of their whole projection and multiplied by ``q_gain`` [heads * dim] / ``k_gain`` [kv_heads * dim]; "head":
@@ -1500,7 +1560,11 @@ def norm_rotary_store(qkv, k_off, v_off, heads, kv_heads, dim, vdim, q_out, q_ga
     ``rot_dims`` entries of every head turn by position * ``inv_freq`` [rot_dims / 2] (float64) in pairs that are
     neighbours (``layout`` "interleaved") or half the rotated entries apart ("half").  Queries go to ``q_out``
     [T, heads * dim]; keys and values to the token's place in the pages (unless ``writes`` is false: then only
-    the queries are made and the pages may be None)."""
+    the queries are made and the pages may be None).  ``taps``: (weights fp32 [columns, taps], state fp32
+    [slots, taps - 1, columns], item_slot, item_start, item_offset, item_count, single_tokens): every column first passes
+    y_t = sum_j w[:, j] u_(t - taps + 1 + j) over the tokens of its request, what lies before this step's portion from the
+    state, which is moved on by this step's rows (in the same kernel where ``single_tokens`` says that every entry
+    brings one token)."""
     _check(qkv, "norm_rotary_store.qkv", torch.float32, 2)
     _check(q_out, "norm_rotary_store.q_out", None, 2)
     _check(inv_freq, "norm_rotary_store.inv_freq", torch.float64, 1)
@@ -1526,12 +1590,29 @@ def norm_rotary_store(qkv, k_off, v_off, heads, kv_heads, dim, vdim, q_out, q_ga
         if (not k_pages.is_contiguous() or not v_pages.is_contiguous() or not block_table.is_contiguous()
                 or k_pages.numel() % (page_size * kv_heads * dim) != 0 or v_pages.numel() % (page_size * kv_heads * vdim) != 0):
             raise KernelError("norm_rotary_store: the pages do not hold whole pages of these rows")
+    tap_args = (None, 0, None, 0, 0, None, None, 0)
+    if taps is not None:
+        weights, state, item_slot, item_start, item_offset, item_count, single = taps
+        _check(weights, "norm_rotary_store.taps", torch.float32, 2)
+        columns, count = weights.shape
+        used = max(heads * dim, k_off + kv_heads * dim if writes else 0, v_off + kv_heads * vdim if writes else 0)
+        if not weights.is_contiguous() or columns > qkv.shape[1] or columns < used:
+            raise KernelError("norm_rotary_store: one row of taps per projected column")
+        if count > 1:
+            _check(state, "norm_rotary_store.state", torch.float32, 3)
+            if tuple(state.shape[1:]) != (count - 1, columns) or state.stride(1) != columns:
+                raise KernelError(f"norm_rotary_store: the state must be [slots, {count - 1}, {columns}]")
+        tap_args = (weights.data_ptr(), count, state.data_ptr() if count > 1 else None, state.stride(0) if count > 1 else 0, columns,
+                    item_slot.data_ptr(), item_start.data_ptr(), int(bool(single)))
     _norm_rotary_store(qkv.data_ptr(), qkv.stride(0), int(k_off), int(v_off), heads, kv_heads, dim, vdim, q_out.data_ptr(),
                        q_out.stride(0), _ptr(q_gain) if mode else None, _ptr(k_gain) if mode and writes else None, mode, float(eps),
                        int(rot_dims), ROTARY_LAYOUTS[layout], inv_freq.data_ptr(), positions.data_ptr(), token_item.data_ptr(),
                        block_table.data_ptr() if writes else None, block_table.shape[1] if writes else 0, page_size,
-                       k_pages.data_ptr() if writes else None, v_pages.data_ptr() if writes else None, int(bool(writes)), n,
-                       dtype_code(q_out.dtype), _stream())
+                       k_pages.data_ptr() if writes else None, v_pages.data_ptr() if writes else None, int(bool(writes)),
+                       *tap_args, n, dtype_code(q_out.dtype), _stream())
+    if taps is not None and count > 1 and not single:
+        _taps_state(state.data_ptr(), state.stride(0), qkv.data_ptr(), qkv.stride(0), item_slot.data_ptr(), item_offset.data_ptr(),
+                    item_count.data_ptr(), item_count.shape[0], columns, count, _stream())
     return q_out
 
 

@@ -15,6 +15,10 @@ the feed-forward are optional roles; the mixer and the feed-forward hand over th
 ``x <- x + norm_2(feed_forward(x))``.  The sublayers read the stream itself, rounded to the activations' type; the
 rounded rows are written by the pass that adds the normed result before them (the first layer rounds by itself).
 
+"parallel_sublayers" has one norm whose output both sublayers read: ``h = norm_1(x)``,
+``x <- x + (mixer(h) + feed_forward(h))``; the feed-forward is optional.  Both add onto the stream in
+place (``h`` lies in a buffer of its own, so neither sees the other's result).
+
 "hyper_connections" is the pre-norm block over several residual streams (``ctx.streams``; see
 ``parts.streams``): each sublayer reads a weighted sum of the streams through its norm and writes
 its result back onto all of them through a mixing matrix.  ``hidden`` is not touched; the model
@@ -101,6 +105,19 @@ class OutputNorm(Arrangement):
             self._add(ctx, parts["norm_2"], hidden, parts["feed_forward"].compute(ctx, self._stream(ctx, hidden)))
 
 
+class ParallelSublayers(Arrangement):
+    roles = ("norm_1", "mixer")
+    optional_roles = ("feed_forward",)               # a layer may have no feed-forward
+
+    def run(self, ctx, parts, hidden, cache):
+        h = parts["norm_1"].forward(ctx, hidden, tag="norm_1")
+        if getattr(cache, "kind", "none") == "composite":
+            cache = cache.sub("mixer")
+        parts["mixer"].forward(ctx, h, hidden, cache)
+        if "feed_forward" in parts:
+            parts["feed_forward"].forward(ctx, h, hidden)
+
+
 class HyperConnections(Arrangement):
     roles = ("streams_1", "norm_1", "mixer")
     optional_roles = ("streams_2", "norm_2", "feed_forward")     # a layer may have no feed-forward
@@ -123,5 +140,6 @@ class HyperConnections(Arrangement):
 
 register_arrangement("pre_norm", PreNorm())
 register_arrangement("output_norm", OutputNorm())
+register_arrangement("parallel_sublayers", ParallelSublayers())
 register_arrangement("hyper_connections", HyperConnections())
 register_arrangement("sandwich_norm", SandwichNorm())

@@ -6,7 +6,7 @@ cached tokens, engine/src/embedding.cu:21-26,100-103).  The head multiplies
 the normed rows whose logits are wanted with the token table itself, without
 bias (engine/src/gpt2.c:245-256); the reference keeps a transposed copy of
 the table for this (engine/src/gpt2_gpu.cu:32-48), here the one [vocab, width]
-table serves the gather and the product.
+table serves the gather and the product.  ``scale`` multiplies the gathered rows (in 32-bit), not the head's.
 """
 
 from __future__ import annotations
@@ -19,9 +19,9 @@ from .spec import WeightSpec
 
 class TokenEmbedding(Embedding):
     graph_safe = True
-    def __init__(self, prefix, vocab_size: int, width: int, name: str = "wte.weight"):
+    def __init__(self, prefix, vocab_size: int, width: int, name: str = "wte.weight", scale: float = 1.0):
         super().__init__(prefix)
-        self.vocab_size, self.width, self.name = int(vocab_size), int(width), name
+        self.vocab_size, self.width, self.name, self.scale = int(vocab_size), int(width), name, float(scale)
 
     def weight_specs(self):
         return [WeightSpec(self.full_name(self.name), (self.vocab_size, self.width), role="table", init="table")]
@@ -29,7 +29,7 @@ class TokenEmbedding(Embedding):
     def forward(self, ctx, position=None):
         hidden = ctx.buffer("hidden", (ctx.n_tokens, self.width), torch.float32)
         table = position.additive_table() if position is not None else None
-        ctx.kernels.embed(hidden, ctx.token_ids, ctx.positions, self.w(self.name), table)
+        ctx.kernels.embed(hidden, ctx.token_ids, ctx.positions, self.w(self.name), table, self.scale)
         if position is not None and table is None:
             position.add_to_hidden(ctx, hidden)
         return hidden

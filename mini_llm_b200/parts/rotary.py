@@ -99,8 +99,9 @@ class BandedRotary(PositionEncoding):
     """Rotary positions on the first ``dims`` entries of every query and key head, pair i turning by
     ``position * f_i``; ``layout`` says which entries form pair i: 2i and 2i+1 ("interleaved") or i and
     i + dims/2 ("half"); the frequencies may be scaled by bands of their wavelength
-    (``banded_frequencies``).  A mixer that norms its queries and keys first calls ``norm_rotate_store``:
-    norm, rotation and the cache store are one kernel."""
+    (``banded_frequencies``).  A mixer whose projections are 32-bit calls ``norm_rotate_store``: a short
+    convolution (``taps``: its weights and state), the queries' and keys' norm, rotation and the cache store are
+    one kernel, the first two optional."""
 
     graph_safe = True
 
@@ -129,11 +130,11 @@ class BandedRotary(PositionEncoding):
         self.inv_freq = torch.tensor(self.frequencies or [0.0], dtype=torch.float64, device=device)
 
     def norm_rotate_store(self, ctx, cache, qkv, q_out, k_off, v_off, n_heads, n_kv_heads, key_size, value_size, q_gain, k_gain,
-                          norm, eps):
+                          norm, eps, taps=None):
         if self.dims > key_size:
             raise ValueError(f"{self.prefix}: {self.dims} rotated entries do not fit a head of {key_size}")
         return ctx.kernels.norm_rotary_store(ctx, cache, qkv, q_out, k_off, v_off, n_heads, n_kv_heads, key_size, value_size,
-                                             q_gain, k_gain, norm, eps, self.dims, self.layout, self.inv_freq)
+                                             q_gain, k_gain, norm, eps, self.dims, self.layout, self.inv_freq, taps)
 
 
 register_part("interleaved_rotary", InterleavedRotary)

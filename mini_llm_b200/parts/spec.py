@@ -110,7 +110,7 @@ class ModelSpec:
 
 @dataclass(frozen=True)
 class PagedKV:
-    """Keys and values of every cached token (or of the last ``window`` tokens; or, with ``block``, of
+    """Keys and values of every cached token (or of the last ``window`` tokens and the first ``keep_first``; or, with ``block``, of
     the tokens of the newest block of that many positions, where queries read keys of their own block
     only), in pages.  With ``has_values`` false only one row per token is kept (the ``keys``): a mixer whose values
     are a part of that row (attention over a shared latent) needs no second pool.  ``value_size``:
@@ -122,6 +122,7 @@ class PagedKV:
     has_values: bool = True
     value_size: int | None = None      # None: as head_size
     block: int | None = None           # None: no blocks; else keys before the newest block of positions are never read again
+    keep_first: int = 0                # with a window: so many first tokens of the sequence are read for ever
 
 
 @dataclass(frozen=True)

@@ -499,7 +499,7 @@ def test_router_with_the_softmax_of_the_chosen_logits():
         pairs = top + (1 if shared else 0)
         choice = torch.zeros(9 * pairs, dtype=torch.int32, device="cuda")
         in_weight, out_weight = torch.zeros(9 * pairs, device="cuda"), torch.zeros(9 * pairs, device="cuda")
-        ops.route(dev(x), dev(router), None, top, choice, in_weight, out_weight, bias=dev(bias), softmax_of_chosen=True, shared_plain=shared)
+        ops.route(dev(x), dev(router), None, top, choice, in_weight, out_weight, bias=dev(bias), rule="softmax_of_chosen", shared_plain=shared)
         logits = x @ router.T + bias
         for t in range(9):
             chosen = np.argsort(-logits[t], kind="stable")[:top]
