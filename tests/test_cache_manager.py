@@ -203,3 +203,32 @@ def test_unreserve_gives_back_what_a_failed_step_took_and_pages_that_go_back_are
     m.close(s)
     assert sum(len(pages) for _, pages in freed) == 3 + 3 + 5 + 5 and m.pages_free() == [6, 6]
     m.check()
+
+
+def test_window_group_keeps_the_first_tokens_pages():
+    """The pages of the first ``keep_first`` tokens stay until the request ends, whether the border of the kept ones
+    lies inside a page or on its edge, and whether fewer tokens than that have come or more are kept than the window sees."""
+    for keep in (1, 8, 11, 70):
+        kept = -(-keep // 8)
+        m = CacheManager([FULL, PagedKV(4, 16, window=20, keep_first=keep), WINDOW], page_size=8, n_pages=[32, 9 + kept, 9], max_requests=2,
+                         max_tokens_per_request=200)
+        freed = []
+        m.on_free = lambda group, pages: freed.extend(pages if group == 1 else [])
+        s = m.open()
+        length = 0
+        for n in [5, 30, 1, 1, 17, 2, 40, 1, 30]:
+            assert m.reserve(s, n), (length, n)
+            m.commit(s, n)
+            length += n
+            m.check()
+            blocks = -(-length // 8)
+            first_needed = max(0, length - 20 + 1) // 8
+            row = m.block_table_row(1, s)
+            held = [b for b in range(blocks) if b < kept or b >= first_needed]
+            assert [b for b in range(len(row)) if row[b] != NO_PAGE] == held and m.pages_held(s)[1] == len(held)
+            assert len(freed) == blocks - len(held)
+            m.unreserve(s)
+            assert m.pages_held(s)[1] == len(held)
+        m.close(s)
+        assert m.pages_free() == [32, 9 + kept, 9] and len(freed) == blocks
+        m.check()

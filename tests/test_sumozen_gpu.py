@@ -198,7 +198,7 @@ def test_bfloat16_follows_within_its_rounding(tmp_path):
     check_rounding(engine, folder, requests, schedule_mixed(requests, {"a": 100, "b": 6, "c": 64}, max_live=3))
     check_rounding(engine, folder, requests, schedule_tail_one_by_one(requests, tail=10))
     chosen = {kernel for key, kernel in engine.kernels.choices.items() if key[0] in ("capped_attention", "linear")}
-    assert {"capped_attention_tiled", "capped_attention_plain", "gemm_tcgen05"} <= chosen
+    assert {"capped_attention_tiled", "split_attention", "gemm_tcgen05"} <= chosen
 
 
 def test_bfloat16_with_sizes_no_fast_kernel_takes(tmp_path):
