@@ -64,13 +64,15 @@ def parse_args():
     parser.add_argument("--kernels", action="store_true",
                         help="time single kernels (matrix products at forced tile widths, prompt attention) back to "
                              "back in a replayed graph and print one line each: the tables of profiles/ come from this")
-    parser.add_argument("--compare", default=None, choices=("fuvolix", "sumozen", "lipulorn", "deluvik"),
+    parser.add_argument("--compare", default=None, choices=("fuvolix", "sumozen", "lipulorn", "deluvik", "nufavik"),
                         help="fuvolix: prefill and decode of Fuvolix stacks at sizes of real layers (random weights), beside "
                              "GPT-2 of equal width, depth and inner size, and their mixers' kernels alone; sumozen: Sumozen "
                              "stacks beside Fuvolix stacks of equal width, depth and inner size, and its kernels alone; "
                              "lipulorn: Lipulorn stacks beside Fuvolix stacks of equal width, depth and feed-forward weights, and "
                              "its kernels alone beside the like kernels of Fuvolix and Sumozen; deluvik: Deluvik stacks beside "
                              "Sumozen stacks of equal width, depth and experts, and its kernels alone beside Sumozen's like kernels; "
+                             "nufavik: Nufavik stacks beside Deluvik stacks of equal width, depth, heads and experts, and its kernels "
+                             "alone beside Deluvik's like kernels; "
                              "one line each")
     parser.add_argument("--tokens-out", default=None,
                         help="(--impl reference) write the greedy tokens of the fixed check workload to this file "
@@ -1468,7 +1470,7 @@ def deluvik_kernels(torch, size: dict, peak: dict):
         choice = torch.zeros(n * pairs, dtype=torch.int32, device="cuda")
         in_weight, out_weight = torch.zeros(n * pairs, device="cuda"), torch.zeros(n * pairs, device="cuda")
         us = replayed_us(torch, lambda i: ops.route(x, router, None, moe["top"], choice, in_weight, out_weight, bias=router_bias,
-                                                    softmax_of_chosen=True, shared_plain=True))
+                                                    rule="softmax_of_chosen", shared_plain=True))
         add(f"router with the softmax of the chosen logits, {name}", us, bytes_moved=n * width * 2.0 + moe["experts"] * width * 2.0)
         us = replayed_us(torch, lambda i: ops.route(x, router, shared_gate, moe["top"], choice, in_weight, out_weight))
         add(f"(Sumozen) router with sigmoid scores, {name}", us, bytes_moved=n * width * 2.0 + (moe["experts"] + 1) * width * 2.0)
@@ -1505,6 +1507,200 @@ def run_compare_deluvik(args):
             print(json.dumps(dict(line, design="deluvik", size=name)), flush=True)
         for line in sumozen_kernels(torch, SUMOZEN_SIZES[size["sumozen"]], peak, recurrences=("mamba",), experts=False):
             print(json.dumps(dict(line, design="sumozen", size=name)), flush=True)
+    return 0
+
+
+# Nufavik stacks beside Deluvik stacks of equal width, depth, heads and experts: every Deluvik layer an "attention_2"
+# (convolved projections, a sink) with routed experts, which have three matrices each there and two here.
+NUFAVIK_SIZES = {
+    "768 wide": {"width": 768, "layers": 12, "attention": {"heads": 12, "kv_heads": 4, "dim": 64, "vdim": 64}, "taps": 4, "window": 512,
+                 "keep_first": 64, "moe": {"experts": 8, "identity": 2, "top": 2, "ff": 768}},
+    "1,024 wide": {"width": 1024, "layers": 24, "attention": {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 96}, "taps": 4, "window": 512,
+                   "keep_first": 64, "moe": {"experts": 8, "identity": 2, "top": 2, "ff": 1024}},
+    "2,048 wide": {"width": 2048, "layers": 16, "attention": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128}, "taps": 4, "window": 512,
+                   "keep_first": 64, "moe": {"experts": 16, "identity": 4, "top": 4, "ff": 1024}},
+}
+
+
+def nufavik_config(size: dict, vocab: int) -> dict:
+    att, moe = size["attention"], size["moe"]
+    layer = {"type": "attention",
+             "mixer": dict(att, conv=size["taps"], scale=att["dim"] ** -0.5, rot={"base": 10000.0, "dims": att["dim"]},
+                           mask={"size": size["window"], "keep_first": size["keep_first"]}),
+             "mlp": {"kind": "moe", "router": {"experts": moe["experts"], "identity": moe["identity"], "top": moe["top"], "scale": 1.5},
+                     "expert": {"ff": moe["ff"]}}}
+    return {"architecture": "Nufavik", "vocab": vocab, "width": size["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "layers": [layer] * size["layers"]}
+
+
+def nufavik_like_config(size: dict, vocab: int) -> dict:
+    att, moe = size["attention"], size["moe"]
+    layer = {"type": "attention_2", "mixer": dict(att, conv=size["taps"], scale=att["dim"] ** -0.5, rot={"base": 10000.0, "dims": att["dim"]}),
+             "mlp": {"kind": "moe", "router": {"experts": moe["experts"], "top": moe["top"]}, "expert": {"ff": moe["ff"]}, "shared": None}}
+    return {"architecture": "Deluvik", "vocab": vocab, "width": size["width"], "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [layer] * size["layers"]}
+
+
+def nufavik_kernels(torch, size: dict, peak: dict):
+    """Nufavik's kernels alone, replayed back to back on operands of their own, each followed by Deluvik's like kernel
+    at the same sizes: prompt portions (2 x 1,024 tokens) and single tokens (8 requests at 1,023 cached tokens), each
+    with the work it must do and the fraction of its bound."""
+    from mini_llm_b200.kernels import ops
+    lines = []
+    page, fma_peak = 64, FP32_FMA_TFLOPS_NOMINAL
+    dev = lambda values: torch.tensor(values, dtype=torch.int32, device="cuda")
+
+    def add(kernel, us, flops=None, bytes_moved=None, tensor_flops=None, **more):
+        line = {"kernel": kernel, "us": round(us, 2), **more}
+        if flops is not None:
+            line.update(tflops=round(flops / us / 1e6, 2), frac_fp32_fma_nominal=round(flops / us / 1e6 / fma_peak, 3))
+        if tensor_flops is not None:
+            line.update(tflops=round(tensor_flops / us / 1e6, 1), frac_bf16_measured=round(tensor_flops / us / 1e6 / peak["bf16_tflops"], 3))
+        if bytes_moved is not None:
+            line.update(gbs=round(bytes_moved / us / 1e3, 1), frac_hbm_measured=round(bytes_moved / us / 1e3 / peak["hbm_gbs"], 3))
+        lines.append(line)
+
+    att, moe, width, taps = size["attention"], size["moe"], size["width"], size["taps"]
+    heads, kv_heads, dim, vdim = att["heads"], att["kv_heads"], att["dim"], att["vdim"]
+    window, keep, scale = size["window"], size["keep_first"], dim ** -0.5
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    for name, lengths, new in (("prompts, 2 x 1024", [1024, 1024], [1024, 1024]), ("single tokens, 8 x 1024", [1024] * 8, [1] * 8)):
+        blocks = [-(-n // page) for n in lengths]
+        table = torch.stack([torch.arange(i * max(blocks), (i + 1) * max(blocks), dtype=torch.int32) for i in range(len(lengths))]).cuda()
+        n, single = sum(new), len(new) > 2
+        starts = [length - count for length, count in zip(lengths, new)]
+        positions = torch.cat([torch.arange(s, s + m) for s, m in zip(starts, new)]).int().cuda()
+        token_item = torch.cat([torch.full((m,), i) for i, m in enumerate(new)]).int().cuda()
+        k_pages = [torch.randn(sum(blocks) + 1, page, kv_heads, dim, device="cuda").bfloat16() for _ in range(4)]
+        v_pages = [torch.randn(sum(blocks) + 1, page, kv_heads, vdim, device="cuda").bfloat16() for _ in range(4)]
+        q = torch.randn(n, heads * dim, device="cuda").bfloat16()
+        out = torch.empty(n, heads * vdim, device="cuda", dtype=torch.bfloat16)
+        sink = torch.zeros(heads, device="cuda")
+        sees = lambda p, w, k: p + 1 if not w else min(p + 1, w) + min(k, max(p + 1 - w, 0))
+        for label, w, kept in ((f"attention within {window} and the first {keep}", window, keep), ("(Deluvik) attention over all keys", 0, 0)):
+            seen = sum(sum(sees(p, w, kept) for p in range(s, s + m)) for s, m in zip(starts, new))
+            if single:
+                chunk, reach = 128, min(table.shape[1] * page, w + kept) if w else table.shape[1] * page
+                chunks, row = -(-reach // chunk), ops.split_attention_row(dim, vdim)
+                scratch = (torch.empty(n * heads * chunks * row, device="cuda"), torch.empty(n * heads * chunks * 2, device="cuda"),
+                           torch.zeros(n * heads, dtype=torch.int32, device="cuda"))
+                us = replayed_us(torch, lambda i: ops.split_attention(out, q, k_pages[i % 4], v_pages[i % 4], table, positions, token_item,
+                                                                      heads, kv_heads, dim, page, scale, w, chunk, chunks, *scratch, sink=sink,
+                                                                      value_size=vdim, keep=kept))
+                add(f"{label}, split keys, {name}", us, bytes_moved=seen * kv_heads * (dim + vdim) * 2.0, heads=heads, kv_heads=kv_heads,
+                    dim=dim, vdim=vdim)
+            else:
+                us = replayed_us(torch, lambda i: ops.capped_attention(out, q, k_pages[i % 4], v_pages[i % 4], table, positions, token_item,
+                                                                       heads, kv_heads, dim, vdim, page, scale, 0.0, w, tiled=True, sink=sink,
+                                                                       keep=kept))
+                add(f"{label}, tiles, {name}", us, flops=2.0 * seen * heads * (dim + vdim), heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim)
+        # taps, rotation and the cache store: reads the 32-bit projections, writes the queries and the pages
+        columns = heads * dim + kv_heads * (dim + vdim)
+        projected = [torch.randn(n, columns, device="cuda") for _ in range(4)]
+        weights = torch.randn(columns, taps, device="cuda")
+        states = [torch.zeros(len(new), taps - 1, columns, device="cuda") for _ in range(4)]
+        q_gain, k_gain = torch.ones(heads * dim, device="cuda"), torch.ones(kv_heads * dim, device="cuda")
+        inv_freq = torch.tensor([10000.0 ** (-2.0 * i / dim) for i in range(dim // 2)], dtype=torch.float64, device="cuda")
+        items = (dev(list(range(len(new)))), dev(starts), dev([sum(new[:i]) for i in range(len(new))]), dev(new))
+        moved = n * columns * 6.0 + 2.0 * len(new) * (taps - 1) * columns * 4
+        for label, norm in (("taps, rotation and cache store", None), ("(Deluvik) taps, norm, rotation and cache store", "whole")):
+            us = replayed_us(torch, lambda i: ops.norm_rotary_store(projected[i % 4], heads * dim, (heads + kv_heads) * dim, heads, kv_heads, dim,
+                                                                    vdim, q, q_gain, k_gain, norm, 1e-5, dim, "half", inv_freq, positions,
+                                                                    token_item, table, page, k_pages[i % 4], v_pages[i % 4],
+                                                                    taps=(weights, states[i % 4], *items, single)))
+            add(f"{label}, {name}", us, bytes_moved=moved, columns=columns, taps=taps)
+        # ---- the router and the experts ----
+        experts, identity, top, inner = moe["experts"], moe["identity"], moe["top"], moe["ff"]
+        x = torch.randn(n, width, device="cuda").bfloat16()
+        hidden = torch.zeros(n, width, device="cuda")
+        router = (torch.randn(experts + identity, width, device="cuda") * 0.05).bfloat16()
+        correction = torch.randn(experts + identity, device="cuda") * 0.02
+        bias = torch.zeros(experts, device="cuda")
+        choice = torch.zeros(n * top, dtype=torch.int32, device="cuda")
+        in_weight, out_weight, passed = torch.zeros(n * top, device="cuda"), torch.zeros(n * top, device="cuda"), torch.zeros(n, device="cuda")
+        total = experts * inner
+        up = [(torch.randn(2 * total, width, device="cuda") * 0.02).bfloat16() for _ in range(4)]
+        down = [(torch.randn(width, total, device="cuda") * 0.02).bfloat16() for _ in range(4)]
+        for gated in (True, False):
+            like = "(Deluvik) " if gated else ""
+            if gated:
+                route = lambda i: ops.route(x, router[:experts], None, top, choice, in_weight, out_weight, bias=bias, rule="softmax_of_chosen")
+            else:
+                route = lambda i: ops.route(x, router, None, top, choice, in_weight, out_weight, rule="softmax_of_all", correction=correction,
+                                            n_identity=identity, scale=1.5, identity_weight=passed)
+            us = replayed_us(torch, route)
+            outputs = experts if gated else experts + identity
+            add(f"{like}router, {name}", us, bytes_moved=(n + outputs) * width * 2.0, outputs=outputs, top=top)
+            pairs = n * top if gated else int((choice >= 0).sum())
+            products = 3 if gated else 2
+            identity_weight = None if gated else passed
+            if single:
+                act = torch.empty(n * top, inner, device="cuda", dtype=torch.bfloat16)
+                tables = []
+                for i in range(4):
+                    place = lambda first: torch.tensor([up[i].data_ptr() + (first + e * inner) * width * 2 for e in range(experts)],
+                                                       dtype=torch.int64, device="cuda")
+                    tables.append((place(0) if gated else None, place(total if gated else 0),
+                                   torch.tensor([down[i].data_ptr() + e * inner * 2 for e in range(experts)], dtype=torch.int64, device="cuda")))
+                inner_of = dev([inner] * experts)
+                us = replayed_us(torch, lambda i: ops.experts(hidden, act, x, choice, in_weight, out_weight, *tables[i % 4], inner_of, inner, top,
+                                                              ld_down=total, identity_weight=identity_weight))
+                used = len(set(choice[choice >= 0].tolist()))
+                add(f"{like}experts, pair by pair, {name}", us, bytes_moved=used * products * inner * width * 2.0, pairs=pairs, experts_used=used)
+            else:
+                gu = torch.empty(n, (2 if gated else 1) * total, device="cuda", dtype=torch.bfloat16)
+                act = torch.empty(n, total, device="cuda", dtype=torch.bfloat16)
+                combine = lambda i: ops.expert_combine(act, gu, choice, in_weight, out_weight, experts, inner, top, top, gated=gated,
+                                                       hidden=hidden, x=x, identity_weight=identity_weight)
+
+                def launch(i):
+                    ops.gemm_bf16(gu, x, up[i % 4][:gu.shape[1]], None, "store", status)
+                    combine(i)
+                    ops.gemm_bf16(hidden, act, down[i % 4], None, "add", status)
+                us = replayed_us(torch, launch)
+                add(f"{like}experts, two products over all experts, {name}", us, tensor_flops=2.0 * pairs * products * width * inner,
+                    executed_tflops=round(2.0 * n * products * width * total / us / 1e6, 1), experts=experts, top=top, inner=inner)
+                us = replayed_us(torch, combine)
+                # reads the chosen experts' columns, writes all of them; the stream for the tokens that pass
+                add(f"{like}activation and weights between the products, {name}", us,
+                    bytes_moved=2.0 * (pairs * inner * (products - 1) + n * total) + (0 if gated else n * width * 10.0))
+        gain = torch.ones(width, device="cuda")
+        streams = [torch.randn(n, width, device="cuda") for _ in range(4)]
+        normed = torch.empty(n, width, device="cuda", dtype=torch.bfloat16)
+        us = replayed_us(torch, lambda i: ops.grouped_rms_norm(normed, streams[i % 4], gain, 1, 1e-5))
+        add(f"norm of the stream, {name}", us, bytes_moved=n * width * (4 + 2.0))
+        us = replayed_us(torch, lambda i: ops.add_normed_cast(streams[i % 4], streams[(i + 1) % 4], gain, 1e-5, normed))
+        add(f"(Deluvik) sum of a normed result with the rounded rows, {name}", us, bytes_moved=n * width * (4 + 4 + 4 + 2.0))
+    return lines
+
+
+def run_compare_nufavik(args):
+    """Nufavik beside Deluvik of equal width, depth, heads and experts: the prompt step of 2,048 tokens (2 x 1,024) and
+    the decode step of ``--batch`` requests at a context of 1,024, in bfloat16, through ``Engine.step``; then the kernels
+    alone, Nufavik's own and Deluvik's like ones.  One JSON line per measurement."""
+    import torch
+    from mini_llm_b200.config import config_from_dict
+    from mini_llm_b200.engine import Engine
+    from mini_llm_b200.weights import write_random_model
+    peak = peaks()
+    context, vocab = 1024, GPT2_SMALL["vocab_size"]
+    for name, size in NUFAVIK_SIZES.items():
+        for design, raw in (("nufavik", nufavik_config(size, vocab)), ("deluvik", nufavik_like_config(size, vocab))):
+            with tempfile.TemporaryDirectory() as folder:
+                write_random_model(config_from_dict(raw), 0, folder, recipe="gpt2", store_dtype="bfloat16")
+                engine = Engine(folder, dtype="bfloat16", max_requests=16, cache_tokens=16 * context, max_tokens_per_step=2048,
+                                **({"page_size": args.page_size} if args.page_size else {}))
+                prefill_ms = prefill_run(engine, 2, 1024, vocab)
+                decode_ms, launches, _ = decode_run(engine, args.batch, args.steps, args.warmup, context, vocab)
+                print(json.dumps({"design": design, "size": name, "width": size["width"], "layers": size["layers"],
+                                  "prefill_2048_tokens_ms": round(prefill_ms, 3), "prefill_tokens_per_s": round(2048 / prefill_ms * 1e3),
+                                  "decode_batch": args.batch, "decode_ms_per_step": round(decode_ms, 3),
+                                  "decode_tokens_per_s": round(args.batch / decode_ms * 1e3), "launches_per_decode_step": launches,
+                                  "weight_bytes": engine.model.weight_bytes, "step_kinds": engine.step_kinds}), flush=True)
+                del engine
+                torch.cuda.empty_cache()
+        for line in nufavik_kernels(torch, size, peak):
+            print(json.dumps(dict(line, size=name)), flush=True)
     return 0
 
 
@@ -1556,6 +1752,8 @@ def main():
         return run_compare_lipulorn(args)
     if args.compare == "deluvik":
         return run_compare_deluvik(args)
+    if args.compare == "nufavik":
+        return run_compare_nufavik(args)
     if args.compare:
         return run_compare(args)
     return run_ours(args)

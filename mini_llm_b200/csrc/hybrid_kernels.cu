@@ -1219,20 +1219,20 @@ extern "C" int mllm_hybrid_linear_recurrence(const RecurrenceParams* params, int
 template <typename T> struct Vec16;
 template <> struct Vec16<float> {
     static constexpr int N = 4;
-    static __device__ __forceinline__ void load(const float* p, float* out) {
-        const float4 v = *reinterpret_cast<const float4*>(p);
-        out[0] = v.x, out[1] = v.y, out[2] = v.z, out[3] = v.w;
+    static __device__ __forceinline__ void unpack(const uint4& v, float* out) {
+        out[0] = __uint_as_float(v.x), out[1] = __uint_as_float(v.y), out[2] = __uint_as_float(v.z), out[3] = __uint_as_float(v.w);
     }
+    static __device__ __forceinline__ void load(const float* p, float* out) { unpack(*reinterpret_cast<const uint4*>(p), out); }
 };
 template <> struct Vec16<bf16> {
     static constexpr int N = 8;
-    static __device__ __forceinline__ void load(const bf16* p, float* out) {
-        const uint4 v = *reinterpret_cast<const uint4*>(p);
+    static __device__ __forceinline__ void unpack(const uint4& v, float* out) {
         out[0] = __uint_as_float(v.x << 16), out[1] = __uint_as_float(v.x & 0xffff0000u);
         out[2] = __uint_as_float(v.y << 16), out[3] = __uint_as_float(v.y & 0xffff0000u);
         out[4] = __uint_as_float(v.z << 16), out[5] = __uint_as_float(v.z & 0xffff0000u);
         out[6] = __uint_as_float(v.w << 16), out[7] = __uint_as_float(v.w & 0xffff0000u);
     }
+    static __device__ __forceinline__ void load(const bf16* p, float* out) { unpack(*reinterpret_cast<const uint4*>(p), out); }
 };
 __device__ __forceinline__ bool aligned16(const void* p) { return (reinterpret_cast<unsigned long long>(p) & 15ull) == 0; }
 static bool aligned_host(const void* p) { return (reinterpret_cast<unsigned long long>(p) & 15ull) == 0; }
@@ -1240,42 +1240,70 @@ static bool aligned_host(const void* p) { return (reinterpret_cast<unsigned long
 // How a token's experts are chosen and weighed (the launcher's `rule`).
 enum RouteRule { ROUTE_SIGMOID_ON_INPUT = 0, ROUTE_SOFTMAX_OF_CHOSEN = 1, ROUTE_SOFTMAX_OF_ALL = 2 };
 
-template <typename T>
-__global__ void __launch_bounds__(128)
+// A block takes TOKENS consecutive tokens (four in long steps: a router row that is read serves all of them) and deals
+// the outputs out to its warps; then a warp a token ranks.
+template <typename T, int TOKENS>
+__global__ void __launch_bounds__(512)
 route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, const float* __restrict__ router_bias,
              const float* __restrict__ correction, const T* __restrict__ shared_gate, int shared_plain, int rule, float scale,
-             int width, int n_outputs, int n_identity, int top, int pairs, int* __restrict__ choice,
+             int width, int n_outputs, int n_identity, int top, int pairs, int n_tokens, int* __restrict__ choice,
              float* __restrict__ in_weight, float* __restrict__ out_weight, float* __restrict__ identity_weight) {
     dependents_may_start();
     wait_for_earlier_kernels();
-    extern __shared__ float shared[];
-    float* row = shared;                       // [width]
-    float* score = row + width;                // [n_outputs + 1]: what ranks the experts
-    float* share = score + n_outputs + 1;      // [n_outputs]: the softmax over all outputs (ROUTE_SOFTMAX_OF_ALL)
-    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) row[c] = to_f32(x[(long)t * ld_x + c]);
+    extern __shared__ __align__(16) float shared[];
+    float* rows = shared;                                  // [TOKENS][width]
+    float* scores = rows + TOKENS * width;                 // [TOKENS][n_outputs + 1]: what ranks the experts
+    float* shares = scores + TOKENS * (n_outputs + 1);     // [TOKENS][n_outputs]: the softmax over all outputs (ROUTE_SOFTMAX_OF_ALL)
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    const int t0 = blockIdx.x * TOKENS, n_here = min(TOKENS, n_tokens - t0);
+    constexpr int N = Vec16<T>::N;
+    const bool vectors = width % N == 0 && aligned16(x) && ld_x % N == 0 && aligned16(router);
+    for (int g = 0; g < TOKENS; g++) {
+        const T* row = x + (long)(t0 + g) * ld_x;
+        if (g >= n_here) {
+            for (int c = threadIdx.x; c < width; c += blockDim.x) rows[g * width + c] = 0.0f;
+        } else if (vectors) {
+            for (int c = threadIdx.x * N; c < width; c += blockDim.x * N) Vec16<T>::load(row + c, rows + g * width + c);
+        } else {
+            for (int c = threadIdx.x; c < width; c += blockDim.x) rows[g * width + c] = to_f32(row[c]);
+        }
+    }
     __syncthreads();
-    for (int e = warp; e < n_outputs + (shared_gate != nullptr ? 1 : 0); e += 4) {
+    for (int e = warp; e < n_outputs + (shared_gate != nullptr ? 1 : 0); e += n_warps) {
         const T* w = e < n_outputs ? router + (long)e * width : shared_gate;
-        float z = 0.0f;
-        constexpr int N = Vec16<T>::N;
-        if (width % N == 0 && aligned16(w)) {
+        float z[TOKENS];
+#pragma unroll
+        for (int g = 0; g < TOKENS; g++) z[g] = 0.0f;
+        if (vectors && aligned16(w)) {
+#pragma unroll 2
             for (int c = lane * N; c < width; c += 32 * N) {
                 float a[N];
                 Vec16<T>::load(w + c, a);
 #pragma unroll
-                for (int i = 0; i < N; i++) z = fmaf(a[i], row[c + i], z);
+                for (int g = 0; g < TOKENS; g++)
+#pragma unroll
+                    for (int i = 0; i < N; i += 4) {
+                        const float4 b = *reinterpret_cast<const float4*>(rows + g * width + c + i);
+                        z[g] = fmaf(a[i], b.x, fmaf(a[i + 1], b.y, fmaf(a[i + 2], b.z, fmaf(a[i + 3], b.w, z[g]))));
+                    }
             }
         } else {
-            for (int c = lane; c < width; c += 32) z = fmaf(to_f32(w[c]), row[c], z);
+            for (int c = lane; c < width; c += 32)
+#pragma unroll
+                for (int g = 0; g < TOKENS; g++) z[g] = fmaf(to_f32(w[c]), rows[g * width + c], z[g]);
         }
-        z = warp_sum(z);
-        if (e < n_outputs && router_bias != nullptr) z += router_bias[e];
-        // (a softmax needs the logits themselves)
-        if (lane == 0) score[e] = rule != ROUTE_SIGMOID_ON_INPUT && e < n_outputs ? z : sigmoid_f(z);
+#pragma unroll
+        for (int g = 0; g < TOKENS; g++) {
+            float sum = warp_sum(z[g]);
+            if (e < n_outputs && router_bias != nullptr) sum += router_bias[e];
+            // (a softmax needs the logits themselves)
+            if (lane == 0) scores[g * (n_outputs + 1) + e] = rule != ROUTE_SIGMOID_ON_INPUT && e < n_outputs ? sum : sigmoid_f(sum);
+        }
     }
     __syncthreads();
-    if (warp != 0) return;
+    if (warp >= n_here) return;
+    const int t = t0 + warp;
+    float *score = scores + warp * (n_outputs + 1), *share = shares + warp * n_outputs;
     // one warp ranks: lane l looks at outputs l, l + 32, ...
     if (rule == ROUTE_SOFTMAX_OF_ALL) {
         float most = -INFINITY, sum = 0.0f;
@@ -1340,27 +1368,26 @@ route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, c
     }
 }
 
-constexpr int UP_FEATURES = 32;                // inner features a block of expert_up takes (four a warp)
-
 // What an expert applies between its two products: silu(gate) * up, or (no gate matrix) the square of relu(up).
 __device__ __forceinline__ float relu_squared(float z) {
     const float r = fmaxf(z, 0.0f);
     return r * r;
 }
 
-template <typename T, bool GATED>
+// A warp takes F inner features of a pair at once: their rows' loads do not wait on one another.
+template <typename T, bool GATED, int F>
 __global__ void __launch_bounds__(256)
 expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long ld_x, const int* __restrict__ choice,
                  const float* __restrict__ in_weight, const long long* __restrict__ gate_of, const long long* __restrict__ up_of,
                  const int* __restrict__ inner_of, int width, int pairs) {
     dependents_may_start();
     wait_for_earlier_kernels();
-    extern __shared__ float row[];             // [width]: the token times its weight, rounded as an activation
+    extern __shared__ __align__(16) float row[];             // [width]: the token times its weight, rounded as an activation
     const int pair = blockIdx.x, t = pair / pairs;
     const int e = choice[pair];
     if (e < 0) return;                         // (an identity expert: expert_down passes the input on)
     const int inner = inner_of[e];
-    const int first = blockIdx.y * UP_FEATURES;
+    const int first = blockIdx.y * 8 * F;
     if (first >= inner) return;
     const float weight = in_weight[pair];
     for (int c = threadIdx.x; c < width; c += blockDim.x)
@@ -1369,35 +1396,51 @@ expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long
     const T* up = (const T*)up_of[e];
     const T* gate = GATED ? (const T*)gate_of[e] : up;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int f = first + warp; f < min(first + UP_FEATURES, inner); f += 8) {
-        const T* g = gate + (long)f * width;
-        const T* u = up + (long)f * width;
-        float zg = 0.0f, zu = 0.0f;
-        constexpr int N = Vec16<T>::N;
-        if (width % N == 0 && aligned16(g) && aligned16(u)) {
-            for (int c = lane * N; c < width; c += 32 * N) {
+    const int f0 = first + warp * F;
+    if (f0 >= inner) return;
+    float zg[F], zu[F];
+#pragma unroll
+    for (int k = 0; k < F; k++) zg[k] = zu[k] = 0.0f;
+    constexpr int N = Vec16<T>::N;
+    if (width % N == 0 && aligned16(gate) && aligned16(up)) {
+        for (int c = lane * N; c < width; c += 32 * N) {
+            uint4 vg[F], vu[F];
+#pragma unroll
+            for (int k = 0; k < F; k++) {
+                const long r = (long)min(f0 + k, inner - 1) * width + c;       // (past the end: the last row once more)
+                if (GATED) vg[k] = *reinterpret_cast<const uint4*>(gate + r);
+                vu[k] = *reinterpret_cast<const uint4*>(up + r);
+            }
+#pragma unroll
+            for (int k = 0; k < F; k++) {
                 float a[N], b[N];
-                if (GATED) Vec16<T>::load(g + c, a);
-                Vec16<T>::load(u + c, b);
+                if (GATED) Vec16<T>::unpack(vg[k], a);
+                Vec16<T>::unpack(vu[k], b);
 #pragma unroll
                 for (int i = 0; i < N; i++) {
-                    if (GATED) zg = fmaf(a[i], row[c + i], zg);
-                    zu = fmaf(b[i], row[c + i], zu);
+                    if (GATED) zg[k] = fmaf(a[i], row[c + i], zg[k]);
+                    zu[k] = fmaf(b[i], row[c + i], zu[k]);
                 }
             }
-        } else {
-            for (int c = lane; c < width; c += 32) {
-                if (GATED) zg = fmaf(to_f32(g[c]), row[c], zg);
-                zu = fmaf(to_f32(u[c]), row[c], zu);
-            }
         }
-        if (GATED) zg = warp_sum(zg);
-        zu = warp_sum(zu);
-        if (lane == 0) act[(long)pair * ld_act + f] = from_f32<T>(GATED ? silu_f(zg) * zu : relu_squared(zu));
+    } else {
+        for (int c = lane; c < width; c += 32)
+#pragma unroll
+            for (int k = 0; k < F; k++) {
+                const long r = (long)min(f0 + k, inner - 1) * width + c;
+                if (GATED) zg[k] = fmaf(to_f32(gate[r]), row[c], zg[k]);
+                zu[k] = fmaf(to_f32(up[r]), row[c], zu[k]);
+            }
+    }
+#pragma unroll
+    for (int k = 0; k < F; k++) {
+        const float g = GATED ? warp_sum(zg[k]) : 0.0f, u = warp_sum(zu[k]);
+        if (lane == 0 && f0 + k < inner) act[(long)pair * ld_act + f0 + k] = from_f32<T>(GATED ? silu_f(g) * u : relu_squared(u));
     }
 }
 
-template <typename T>
+// A warp takes C columns of a token's sum: every pair's loads of all of them are asked for together.
+template <typename T, int C>
 __global__ void __launch_bounds__(256)
 expert_down_kernel(float* __restrict__ hidden, long ld_hidden, const T* __restrict__ act, long ld_act,
                    const int* __restrict__ choice, const float* __restrict__ out_weight, const long long* __restrict__ down_of,
@@ -1406,33 +1449,55 @@ expert_down_kernel(float* __restrict__ hidden, long ld_hidden, const T* __restri
     dependents_may_start();
     wait_for_earlier_kernels();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int c = blockIdx.y * 8 + warp; c < width; c += gridDim.y * 8) {
-        float total = 0.0f;
-        for (int k = 0; k < pairs; k++) {
-            const long pair = (long)t * pairs + k;
-            const int e = choice[pair];
-            if (e < 0) continue;
-            const int inner = inner_of[e];
-            const T* w = (const T*)down_of[e] + (long)c * ld_down;
-            const T* a = act + pair * ld_act;
-            float z = 0.0f;
-            constexpr int N = Vec16<T>::N;
-            if (inner % N == 0 && aligned16(w) && aligned16(a)) {
-                for (int f = lane * N; f < inner; f += 32 * N) {
-                    float x[N], y[N];
-                    Vec16<T>::load(w + f, x);
-                    Vec16<T>::load(a + f, y);
+    const int c0 = (blockIdx.y * 8 + warp) * C;
+    if (c0 >= width) return;
+    constexpr int N = Vec16<T>::N;
+    float total[C];
 #pragma unroll
-                    for (int i = 0; i < N; i++) z = fmaf(x[i], y[i], z);
+    for (int q = 0; q < C; q++) total[q] = 0.0f;
+#pragma unroll 2
+    for (int k = 0; k < pairs; k++) {
+        const long pair = (long)t * pairs + k;
+        const int e = choice[pair];
+        if (e < 0) continue;
+        const int inner = inner_of[e];
+        const T* w = (const T*)down_of[e];
+        const T* a = act + pair * ld_act;
+        float z[C];
+#pragma unroll
+        for (int q = 0; q < C; q++) z[q] = 0.0f;
+        if (inner % N == 0 && ld_down % N == 0 && aligned16(w) && aligned16(a)) {
+#pragma unroll 2
+            for (int f = lane * N; f < inner; f += 32 * N) {
+                uint4 v[C];
+#pragma unroll
+                for (int q = 0; q < C; q++) v[q] = *reinterpret_cast<const uint4*>(w + (long)min(c0 + q, width - 1) * ld_down + f);
+                float y[N];
+                Vec16<T>::load(a + f, y);
+#pragma unroll
+                for (int q = 0; q < C; q++) {
+                    float b[N];
+                    Vec16<T>::unpack(v[q], b);
+#pragma unroll
+                    for (int i = 0; i < N; i++) z[q] = fmaf(b[i], y[i], z[q]);
                 }
-            } else {
-                for (int f = lane; f < inner; f += 32) z = fmaf(to_f32(w[f]), to_f32(a[f]), z);
             }
-            total = fmaf(out_weight[pair], warp_sum(z), total);
+        } else {
+            for (int f = lane; f < inner; f += 32)
+#pragma unroll
+                for (int q = 0; q < C; q++) z[q] = fmaf(to_f32(w[(long)min(c0 + q, width - 1) * ld_down + f]), to_f32(a[f]), z[q]);
         }
+#pragma unroll
+        for (int q = 0; q < C; q++) total[q] = fmaf(out_weight[pair], warp_sum(z[q]), total[q]);
+    }
+#pragma unroll
+    for (int q = 0; q < C; q++) {
+        const int c = c0 + q;
+        if (lane != 0 || c >= width) continue;
         // identity experts hand the token on as it came
-        if (identity_weight != nullptr) total = fmaf(identity_weight[t], to_f32(x[(long)t * ld_x + c]), total);
-        if (lane == 0) hidden[(long)t * ld_hidden + c] = assign ? total : hidden[(long)t * ld_hidden + c] + total;
+        if (identity_weight != nullptr) total[q] = fmaf(identity_weight[t], to_f32(x[(long)t * ld_x + c]), total[q]);
+        float* h = hidden + (long)t * ld_hidden + c;
+        *h = assign ? total[q] : *h + total[q];
     }
 }
 
@@ -1547,14 +1612,18 @@ extern "C" int mllm_hybrid_route(const void* x, long ld_x, const void* router, c
         return fail("route: identity experts need weights on the outputs and room for the token's sum of them");
     cudaStream_t s = (cudaStream_t)stream;
     const int pairs = top + (shared_gate != nullptr || shared_plain ? 1 : 0);
-    const size_t shared = sizeof(float) * ((size_t)width + 2 * (size_t)n_outputs + 1);
-    if (shared > 48 * 1024) return fail("route: the token and the scores do not fit shared memory");
-#define RUN(T)                                                                                                                  \
-    launch_kernel(g_dependent_launch != 0, route_kernel<T>, dim3(n_tokens), dim3(128), shared, s, (const T*)x, ld_x,            \
-                  (const T*)router, router_bias, correction, (const T*)shared_gate, shared_plain, rule, scale, width, n_outputs, \
-                  n_identity, top, pairs, choice, in_weight, out_weight, identity_weight)
-    if (dtype == DT_F32) RUN(float);
-    else if (dtype == DT_BF16) RUN(bf16);
+    const size_t one = sizeof(float) * ((size_t)width + 2 * (size_t)n_outputs + 1);
+    if (one > 48 * 1024) return fail("route: the token and the scores do not fit shared memory");
+    const bool four = n_tokens >= 512 && 4 * one <= 48 * 1024;
+    // a warp for every output in steps of few tokens, four to sixteen of them
+    const int warps = four ? 8 : (n_tokens >= 512 || n_outputs <= 4 ? 4 : (n_outputs < 16 ? n_outputs : 16));
+#define RUN(T, TOKENS)                                                                                                          \
+    launch_kernel(g_dependent_launch != 0, route_kernel<T, TOKENS>, dim3((n_tokens + TOKENS - 1) / TOKENS), dim3(32 * warps),   \
+                  TOKENS * one, s, (const T*)x, ld_x, (const T*)router, router_bias, correction, (const T*)shared_gate,         \
+                  shared_plain, rule, scale, width, n_outputs, n_identity, top, pairs, n_tokens, choice, in_weight, out_weight, \
+                  identity_weight)
+    if (dtype == DT_F32) { if (four) RUN(float, 4); else RUN(float, 1); }
+    else if (dtype == DT_BF16) { if (four) RUN(bf16, 4); else RUN(bf16, 1); }
     else return fail("route: unknown dtype");
 #undef RUN
     return check_launch("route_kernel");
@@ -1570,20 +1639,18 @@ extern "C" int mllm_hybrid_experts(float* hidden, long ld_hidden, void* act, lon
     cudaStream_t s = (cudaStream_t)stream;
     const size_t shared = sizeof(float) * (size_t)width;
     if (shared > 48 * 1024) return fail("experts: the token does not fit shared memory");
-    dim3 up_grid(n_tokens * pairs, (max_inner + UP_FEATURES - 1) / UP_FEATURES);
-    if (up_grid.y > 65535) return fail("experts: the inner size is too large for one launch");
-    int down_y = (width + 7) / 8;
-    if (down_y > 16) down_y = 16;
-    dim3 down_grid(n_tokens, down_y);
+    constexpr int F = 4, C = 2;
+    dim3 up_grid(n_tokens * pairs, (max_inner + 8 * F - 1) / (8 * F)), down_grid(n_tokens, (width + 8 * C - 1) / (8 * C));
+    if (up_grid.y > 65535 || down_grid.y > 65535) return fail("experts: the sizes are too large for one launch");
 #define RUN(T)                                                                                                                  \
     do {                                                                                                                        \
         if (gate_of != nullptr)                                                                                                 \
-            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, true>, up_grid, dim3(256), shared, s, (T*)act, ld_act,   \
+            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, true, F>, up_grid, dim3(256), shared, s, (T*)act, ld_act, \
                           (const T*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);                        \
         else                                                                                                                    \
-            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, false>, up_grid, dim3(256), shared, s, (T*)act, ld_act,  \
+            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, false, F>, up_grid, dim3(256), shared, s, (T*)act, ld_act, \
                           (const T*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);                        \
-        launch_kernel(g_dependent_launch != 0, expert_down_kernel<T>, down_grid, dim3(256), 0, s, hidden, ld_hidden,            \
+        launch_kernel(g_dependent_launch != 0, expert_down_kernel<T, C>, down_grid, dim3(256), 0, s, hidden, ld_hidden,         \
                       (const T*)act, ld_act, choice, out_weight, down_of, inner_of, ld_down, width, pairs, assign, (const T*)x, \
                       ld_x, identity_weight);                                                                                   \
     } while (0)

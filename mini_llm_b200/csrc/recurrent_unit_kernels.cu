@@ -33,108 +33,239 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + l
 // lies before this step's portion comes from the request's `tap_state` (the last taps - 1 projected rows, oldest
 // first, 32-bit), which a step of single tokens (tap_moves) also moves on here, each column by the one thread that
 // reads it; after other steps a pass of its own does (another block may still need the rows).
-// One block per token; the token's q and k lie in shared memory in 32-bit.
+// A block takes G consecutive tokens (4 in steps with prompt portions: a column's taps are read once and a row's
+// entry serves up to `taps` of the block's tokens; 1 in steps of single tokens) and `heads_per_block` of the query and
+// key heads side by side (all of them where the norm is over the whole projection), a key head with its value head.
+// Its q and k lie in shared memory in 32-bit.
 // ---------------------------------------------------------------------------
-template <typename T>
-__global__ void __launch_bounds__(256)
-norm_rotary_store_kernel(const float* __restrict__ qkv, long ld, int k_off, int v_off, int heads, int kv_heads, int dim,
-                         int vdim, T* __restrict__ q_out, long ld_q, const float* __restrict__ q_gain,
-                         const float* __restrict__ k_gain, int norm_mode, float eps, int rot_dims, int layout,
-                         const double* __restrict__ inv_freq, const int* __restrict__ positions,
-                         const int* __restrict__ token_item, const int* __restrict__ block_table, int max_blocks,
-                         int page_size, T* __restrict__ k_pages, T* __restrict__ v_pages, int writes,
-                         const float* __restrict__ tap_weights, int taps, float* tap_state, long tap_stride, int tap_width,
-                         const int* __restrict__ item_slot, const int* __restrict__ item_start, int tap_moves) {
+struct NormRotaryParams {
+    const float* qkv;
+    long ld;
+    int k_off, v_off, heads, kv_heads, dim, vdim;
+    void* q_out;
+    long ld_q;
+    const float *q_gain, *k_gain;
+    int norm_mode;
+    float eps;
+    int rot_dims, layout;
+    const double* inv_freq;
+    const int *positions, *token_item, *block_table;
+    int max_blocks, page_size;
+    void *k_pages, *v_pages;
+    int writes;
+    const float* tap_weights;
+    int taps;
+    float* tap_state;
+    long tap_stride;
+    int tap_width;
+    const int *item_slot, *item_start;
+    int tap_moves;
+    int n_tokens, heads_per_block;
+};
+
+// cosine and sine of position * f: the angle in 64-bit, brought into [-pi, pi] there and split into a 32-bit value
+// and what its rounding left, which enters in first order.
+__device__ __forceinline__ void turn_of(int position, double f, float* c, float* s) {
+    const double angle = (double)position * f;
+    const double r = fma(-rint(angle * 0.15915494309189535), 6.283185307179586, angle);
+    const float hi = (float)r, lo = (float)(r - (double)hi);
+    float sh, ch;
+    sincosf(hi, &sh, &ch);
+    *c = fmaf(-lo, sh, ch);
+    *s = fmaf(lo, ch, sh);
+}
+
+// TAPS: 0 none, 1 .. 4 as given, -1 read from the parameters
+template <typename T, int G, int TAPS>
+__global__ void __launch_bounds__(G > 1 ? 256 : 1024)
+norm_rotary_store_kernel(NormRotaryParams pp) {
     dependents_may_start();
     wait_for_earlier_kernels();
     extern __shared__ float shared[];
-    const int all_heads = heads + (writes ? kv_heads : 0);
-    const int half = rot_dims / 2;
-    float* turn = shared;                       // [rot_dims / 2][2]: cosine, sine
-    float* inverse = turn + 2 * half + 2;       // [all_heads]: 1 / root mean square of the head's norm group
-    float* scratch = inverse + all_heads;       // [33]
-    float* x = scratch + 33;                    // [all_heads * dim]: q heads, then k heads
-    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
-    const int p = positions[t];
-    const float* row = qkv + (long)t * ld;
-    const int item = token_item[t];
-    const int local = taps > 1 ? p - item_start[item] : 0;          // tokens of this request before t in this step
-    float* held = taps > 1 ? tap_state + (long)item_slot[item] * tap_stride : nullptr;
-    auto column = [&](int c) {
-        const float mine = row[c];
-        if (taps <= 0) return mine;
-        const float* w = tap_weights + (long)c * taps;
-        float acc = 0.0f;
-        for (int back = taps - 1; back >= 1; back--) {
-            const float v = local >= back ? row[c - (long)back * ld] : held[(long)(taps - 1 + local - back) * tap_width + c];
-            acc = fmaf(w[taps - 1 - back], v, acc);
-        }
-        acc = fmaf(w[taps - 1], mine, acc);
-        if (tap_moves && taps > 1) {
-            for (int s = 0; s + 1 < taps - 1; s++) held[(long)s * tap_width + c] = held[(long)(s + 1) * tap_width + c];
-            held[(long)(taps - 2) * tap_width + c] = mine;
-        }
-        return acc;
-    };
-    for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        double s, c;
-        sincos((double)p * inv_freq[i], &s, &c);
-        turn[2 * i] = (float)c;
-        turn[2 * i + 1] = (float)s;
-    }
-    const int q_width = heads * dim, k_width = kv_heads * dim;
-    for (int c = threadIdx.x; c < q_width; c += blockDim.x) x[c] = column(c);
-    long slot = 0;
-    if (writes) {
-        slot = (long)block_table[(long)item * max_blocks + p / page_size] * page_size + (p % page_size);
-        for (int c = threadIdx.x; c < k_width; c += blockDim.x) x[q_width + c] = column(k_off + c);
-        // the values leave first: they may be the keys as projected (then the thread that filtered a column has it)
-        for (int c = threadIdx.x; c < kv_heads * vdim; c += blockDim.x)
-            v_pages[slot * kv_heads * vdim + c] = from_f32<T>(v_off == k_off ? x[q_width + c] : column(v_off + c));
+    __shared__ int tok_pos[G], tok_local[G], tok_slot[G];
+    __shared__ long tok_place[G];
+    const int dim = pp.dim, half = pp.rot_dims / 2;
+    const int all_heads = pp.heads + (pp.writes ? pp.kv_heads : 0);
+    const int h0 = blockIdx.y * pp.heads_per_block, nh = min(pp.heads_per_block, all_heads - h0);
+    const int t0 = blockIdx.x * G, n_here = min(G, pp.n_tokens - t0);
+    float* turn = shared;                                 // [G][half][2]: cosine, sine
+    float* inverse = turn + 2 * G * half;                 // [G][heads_per_block]: 1 / root mean square of the head's norm group
+    float* scratch = inverse + G * pp.heads_per_block;    // [33]
+    float* x = scratch + 33;                              // [G][heads_per_block * dim]: the block's heads
+    const int xs = pp.heads_per_block * dim;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    const bool filters = TAPS != 0 && (TAPS > 1 || pp.taps > 1);       // (one tap scales the row itself)
+    if (threadIdx.x < n_here) {
+        const int t = t0 + threadIdx.x, p = pp.positions[t], item = pp.token_item[t];
+        tok_pos[threadIdx.x] = p;
+        tok_local[threadIdx.x] = filters ? p - pp.item_start[item] : 0;        // tokens of this request before t in this step
+        tok_slot[threadIdx.x] = filters ? pp.item_slot[item] : 0;
+        if (pp.writes)
+            tok_place[threadIdx.x] = (long)pp.block_table[(long)item * pp.max_blocks + p / pp.page_size] * pp.page_size + (p % pp.page_size);
     }
     __syncthreads();
-    if (norm_mode == 1) {
-        float sq = 0.0f, sk = 0.0f;
-        for (int c = threadIdx.x; c < q_width; c += blockDim.x) sq = fmaf(x[c], x[c], sq);
-        if (writes)
-            for (int c = threadIdx.x; c < k_width; c += blockDim.x) sk = fmaf(x[q_width + c], x[q_width + c], sk);
-        sq = block_sum(sq, scratch);
-        if (writes) sk = block_sum(sk, scratch);
-        const float iq = 1.0f / sqrtf(sq / (float)q_width + eps), ik = writes ? 1.0f / sqrtf(sk / (float)k_width + eps) : 0.0f;
-        for (int h = threadIdx.x; h < all_heads; h += blockDim.x) inverse[h] = h < heads ? iq : ik;
-    } else {
-        for (int h = warp; h < all_heads; h += n_warps) {
-            float s = 0.0f;
-            if (norm_mode == 2)
-                for (int d = lane; d < dim; d += 32) s = fmaf(x[h * dim + d], x[h * dim + d], s);
-            s = warp_sum(s);
-            if (lane == 0) inverse[h] = norm_mode == 2 ? 1.0f / sqrtf(s / (float)dim + eps) : 1.0f;
-        }
-    }
-    __syncthreads();
-    // a unit of work: one pair of the rotated part, or one entry of what passes unchanged
-    const int units = half + (dim - rot_dims);
-    for (int u = threadIdx.x; u < all_heads * units; u += blockDim.x) {
-        const int h = u / units, j = u % units;
-        const bool is_key = h >= heads;
-        const float* gain = is_key ? k_gain : q_gain;
-        const int gain_base = norm_mode == 1 ? (is_key ? h - heads : h) * dim : 0;
-        const float inv = inverse[h];
-        T* dst = is_key ? k_pages + (slot * kv_heads + (h - heads)) * dim : q_out + (long)t * ld_q + (long)h * dim;
-        if (j < half) {
-            const int ia = layout == 0 ? 2 * j : j, ib = layout == 0 ? 2 * j + 1 : j + half;
-            float a = x[h * dim + ia] * inv, b = x[h * dim + ib] * inv;
-            if (norm_mode != 0) a *= gain[gain_base + ia], b *= gain[gain_base + ib];
-            const float c = turn[2 * j], s = turn[2 * j + 1];
-            dst[ia] = from_f32<T>(a * c - b * s);
-            dst[ib] = from_f32<T>(b * c + a * s);
+
+    // column c of the block's tokens, filtered
+    auto column = [&](int c, float* y) {
+        const float* base = pp.qkv + c;
+        if (TAPS == 0) {
+#pragma unroll
+            for (int g = 0; g < G; g++) y[g] = g < n_here ? base[(long)(t0 + g) * pp.ld] : 0.0f;
+        } else if (TAPS > 0) {
+            constexpr int TP = TAPS > 0 ? TAPS : 1;
+            float u[G + TP - 1], w[TP];
+#pragma unroll
+            for (int i = 0; i < G + TP - 1; i++) {
+                const int r = t0 - (TP - 1) + i;
+                u[i] = r >= 0 && r < t0 + n_here && (i >= TP - 1 || !pp.tap_moves) ? base[(long)r * pp.ld] : 0.0f;
+            }
+            if (TP == 4) {
+                const float4 v = *reinterpret_cast<const float4*>(pp.tap_weights + (long)c * TP);
+                w[0] = v.x, w[1 % TP] = v.y, w[2 % TP] = v.z, w[3 % TP] = v.w;
+            } else {
+#pragma unroll
+                for (int j = 0; j < TP; j++) w[j] = pp.tap_weights[(long)c * TP + j];
+            }
+#pragma unroll
+            for (int g = 0; g < G; g++) {
+                y[g] = 0.0f;
+                if (g >= n_here) continue;
+                const int local = tok_local[g];
+                float* held = TP > 1 ? pp.tap_state + (long)tok_slot[g] * pp.tap_stride + c : nullptr;
+                float past[TP];
+#pragma unroll
+                for (int j = 0; j + 1 < TP; j++)           // (entry local + j of the state, where the step itself does not reach back)
+                    past[j] = local >= TP - 1 - j ? u[g + j] : held[(long)(local + j) * pp.tap_width];
+                past[TP - 1] = u[g + TP - 1];
+#pragma unroll
+                for (int j = 0; j < TP; j++) y[g] = fmaf(w[j], past[j], y[g]);
+                if (G == 1 && pp.tap_moves) {
+#pragma unroll
+                    for (int j = 0; j + 1 < TP; j++) held[(long)j * pp.tap_width] = past[j + 1];
+                }
+            }
         } else {
-            const int d = rot_dims + (j - half);
-            float a = x[h * dim + d] * inv;
-            if (norm_mode != 0) a *= gain[gain_base + d];
-            dst[d] = from_f32<T>(a);
+            const int taps = pp.taps;
+            const float* w = pp.tap_weights + (long)c * taps;
+            for (int g = 0; g < n_here; g++) {
+                const int local = tok_local[g];
+                float* held = taps > 1 ? pp.tap_state + (long)tok_slot[g] * pp.tap_stride + c : nullptr;
+                const float mine = base[(long)(t0 + g) * pp.ld];
+                float acc = 0.0f;
+                for (int back = taps - 1; back >= 1; back--) {
+                    const float v = local >= back ? base[(long)(t0 + g - back) * pp.ld] : held[(long)(taps - 1 + local - back) * pp.tap_width];
+                    acc = fmaf(w[taps - 1 - back], v, acc);
+                }
+                y[g] = fmaf(w[taps - 1], mine, acc);
+                if (pp.tap_moves && taps > 1) {
+                    for (int s = 0; s + 1 < taps - 1; s++) held[(long)s * pp.tap_width] = held[(long)(s + 1) * pp.tap_width];
+                    held[(long)(taps - 2) * pp.tap_width] = mine;
+                }
+            }
+        }
+    };
+
+    const int q_width = pp.heads * dim;
+    for (int lc = threadIdx.x; lc < nh * dim; lc += blockDim.x) {
+        const int at = h0 * dim + lc;
+        float y[G];
+        column(at < q_width ? at : pp.k_off + (at - q_width), y);
+#pragma unroll
+        for (int g = 0; g < G; g++)
+            if (g < n_here) x[g * xs + lc] = y[g];
+    }
+    const int first_key = max(h0, pp.heads) - pp.heads, n_keys = pp.writes ? h0 + nh - pp.heads - first_key : 0;   // key heads of this block
+    T* v_pages = (T*)pp.v_pages;
+    const long v_row = (long)pp.kv_heads * pp.vdim;
+    if (n_keys > 0 && pp.v_off != pp.k_off)
+        for (int i = threadIdx.x; i < n_keys * pp.vdim; i += blockDim.x) {
+            const int at = first_key * pp.vdim + i;
+            float y[G];
+            column(pp.v_off + at, y);
+#pragma unroll
+            for (int g = 0; g < G; g++)
+                if (g < n_here) v_pages[tok_place[g] * v_row + at] = from_f32<T>(y[g]);
+        }
+    for (int i = threadIdx.x; i < half * n_here; i += blockDim.x)
+        turn_of(tok_pos[i / half], pp.inv_freq[i % half], &turn[2 * i], &turn[2 * i + 1]);
+    __syncthreads();
+    if (n_keys > 0 && pp.v_off == pp.k_off) {
+        // values that are the keys as they came in
+        const int from = (pp.heads + first_key - h0) * dim;
+        for (int g = 0; g < n_here; g++)
+            for (int i = threadIdx.x; i < n_keys * dim; i += blockDim.x)
+                v_pages[tok_place[g] * v_row + first_key * dim + i] = from_f32<T>(x[g * xs + from + i]);
+    }
+    if (pp.norm_mode == 1) {
+        const int k_width = pp.kv_heads * dim;
+        for (int g = 0; g < n_here; g++) {
+            float sq = 0.0f, sk = 0.0f;
+            for (int c = threadIdx.x; c < q_width; c += blockDim.x) sq = fmaf(x[g * xs + c], x[g * xs + c], sq);
+            if (pp.writes)
+                for (int c = threadIdx.x; c < k_width; c += blockDim.x) sk = fmaf(x[g * xs + q_width + c], x[g * xs + q_width + c], sk);
+            sq = block_sum(sq, scratch);
+            if (pp.writes) sk = block_sum(sk, scratch);
+            const float iq = 1.0f / sqrtf(sq / (float)q_width + pp.eps), ik = pp.writes ? 1.0f / sqrtf(sk / (float)k_width + pp.eps) : 0.0f;
+            for (int h = threadIdx.x; h < nh; h += blockDim.x) inverse[g * pp.heads_per_block + h] = h < pp.heads ? iq : ik;
+        }
+        __syncthreads();
+    }
+    // a warp takes a token's head; its units of work: the pairs of the rotated part, then the entries that pass unchanged
+    const int units = half + (dim - pp.rot_dims);
+    for (int r = warp; r < n_here * nh; r += n_warps) {
+        const int g = r / nh, lh = r % nh, h = h0 + lh;
+        const bool is_key = h >= pp.heads;
+        const float* row = x + g * xs + lh * dim;
+        float inv = 1.0f;
+        if (pp.norm_mode == 1) inv = inverse[g * pp.heads_per_block + lh];
+        if (pp.norm_mode == 2) {
+            float sum = 0.0f;
+            for (int d = lane; d < dim; d += 32) sum = fmaf(row[d], row[d], sum);
+            inv = 1.0f / sqrtf(warp_sum(sum) / (float)dim + pp.eps);
+        }
+        const float* gain = pp.norm_mode == 0 ? nullptr : (is_key ? pp.k_gain : pp.q_gain) + (pp.norm_mode == 1 ? (is_key ? h - pp.heads : h) * dim : 0);
+        T* dst = is_key ? (T*)pp.k_pages + (tok_place[g] * pp.kv_heads + (h - pp.heads)) * dim
+                        : (T*)pp.q_out + (long)(t0 + g) * pp.ld_q + (long)h * dim;
+        for (int j = lane; j < units; j += 32) {
+            if (j < half) {
+                const int ia = pp.layout == 0 ? 2 * j : j, ib = pp.layout == 0 ? 2 * j + 1 : j + half;
+                float a = row[ia] * inv, b = row[ib] * inv;
+                if (gain != nullptr) a *= gain[ia], b *= gain[ib];
+                const float c = turn[2 * (g * half + j)], s = turn[2 * (g * half + j) + 1];
+                dst[ia] = from_f32<T>(a * c - b * s);
+                dst[ib] = from_f32<T>(b * c + a * s);
+            } else {
+                const int d = pp.rot_dims + (j - half);
+                float a = row[d] * inv;
+                if (gain != nullptr) a *= gain[d];
+                dst[d] = from_f32<T>(a);
+            }
         }
     }
+}
+
+template <typename T, int G, int TAPS>
+static int launch_norm_rotary(const NormRotaryParams& pp, int threads, size_t shared, cudaStream_t s) {
+    if (shared > 48 * 1024 &&
+        cudaFuncSetAttribute(norm_rotary_store_kernel<T, G, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared) != cudaSuccess)
+        return fail("norm_rotary_store: the shared memory was refused");
+    const int all_heads = pp.heads + (pp.writes ? pp.kv_heads : 0);
+    dim3 grid((pp.n_tokens + G - 1) / G, (all_heads + pp.heads_per_block - 1) / pp.heads_per_block);
+    launch_kernel(g_dependent_launch != 0, norm_rotary_store_kernel<T, G, TAPS>, grid, dim3(threads), shared, s, pp);
+    return check_launch("norm_rotary_store_kernel");
+}
+
+template <typename T, int G>
+static int pick_norm_rotary(const NormRotaryParams& pp, int threads, size_t shared, cudaStream_t s) {
+    const bool aligned = (reinterpret_cast<unsigned long long>(pp.tap_weights) & 15ull) == 0;
+    switch (pp.taps) {
+    case 0: return launch_norm_rotary<T, G, 0>(pp, threads, shared, s);
+    case 2: return launch_norm_rotary<T, G, 2>(pp, threads, shared, s);
+    case 3: return launch_norm_rotary<T, G, 3>(pp, threads, shared, s);
+    case 4: if (aligned) return launch_norm_rotary<T, G, 4>(pp, threads, shared, s); break;
+    default: break;
+    }
+    return launch_norm_rotary<T, G, -1>(pp, threads, shared, s);
 }
 
 extern "C" int mllm_unit_norm_rotary_store(const float* qkv, long ld, int k_off, int v_off, int heads, int kv_heads, int dim,
@@ -153,25 +284,24 @@ extern "C" int mllm_unit_norm_rotary_store(const float* qkv, long ld, int k_off,
     if (taps < 0 || (taps > 1 && (tap_state == nullptr || item_slot == nullptr || item_start == nullptr)))
         return fail("norm_rotary_store: taps need the requests' last rows");
     if (writes && v_off == k_off && vdim != dim) return fail("norm_rotary_store: values that are the keys have their size");
-    cudaStream_t s = (cudaStream_t)stream;
     const int all_heads = heads + (writes ? kv_heads : 0);
-    const size_t shared = sizeof(float) * ((size_t)rot_dims + 2 + all_heads + 33 + (size_t)all_heads * dim);
-    if (shared > 200 * 1024) return fail("norm_rotary_store: a token's queries and keys do not fit shared memory");
-#define RUN(T)                                                                                                                   \
-    do {                                                                                                                         \
-        if (shared > 48 * 1024 &&                                                                                                \
-            cudaFuncSetAttribute(norm_rotary_store_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)shared) != cudaSuccess) \
-            return fail("norm_rotary_store: the shared memory was refused");                                                     \
-        launch_kernel(g_dependent_launch != 0, norm_rotary_store_kernel<T>, dim3(n_tokens), dim3(256), shared, s, qkv, ld, k_off, \
-                      v_off, heads, kv_heads, dim, vdim, (T*)q_out, ld_q, q_gain, k_gain, norm_mode, eps, rot_dims, layout,      \
-                      inv_freq, positions, token_item, block_table, max_blocks, page_size, (T*)k_pages, (T*)v_pages, writes,     \
-                      tap_weights, taps, tap_state, tap_stride, tap_width, item_slot, item_start, tap_moves);                    \
-    } while (0)
-    if (dtype == DT_F32) RUN(float);
-    else if (dtype == DT_BF16) RUN(bf16);
-    else return fail("norm_rotary_store: unknown dtype");
-#undef RUN
-    return check_launch("norm_rotary_store_kernel");
+    // one token a block where every entry brings one (the state moves with it) and in short steps, else four; as many
+    // heads a block as give its threads a few columns each, all of them where a norm spans them
+    int group = tap_moves || n_tokens < 64 ? 1 : 4;
+    int per_block = (group == 4 ? 1024 : 256) / dim;
+    per_block = norm_mode == 1 ? all_heads : (per_block < 1 ? 1 : (per_block > all_heads ? all_heads : per_block));
+    auto bytes = [&](int g) { return sizeof(float) * ((size_t)g * (rot_dims + per_block + (size_t)per_block * dim) + 33); };
+    if (group == 4 && bytes(4) > 96 * 1024) group = 1;
+    if (bytes(group) > 200 * 1024) return fail("norm_rotary_store: a token's queries and keys do not fit shared memory");
+    const NormRotaryParams pp = {qkv, ld, k_off, v_off, heads, kv_heads, dim, vdim, q_out, ld_q, q_gain, k_gain, norm_mode, eps, rot_dims,
+                                 layout, inv_freq, positions, token_item, block_table, max_blocks, page_size, k_pages, v_pages, writes,
+                                 tap_weights, taps, tap_state, tap_stride, tap_width, item_slot, item_start, tap_moves, n_tokens, per_block};
+    cudaStream_t s = (cudaStream_t)stream;
+    int threads = 256;
+    if (group == 1 && per_block * dim >= 1024) threads = per_block * dim >= 2048 ? 1024 : 512;
+    if (dtype == DT_F32) return group == 4 ? pick_norm_rotary<float, 4>(pp, threads, bytes(4), s) : pick_norm_rotary<float, 1>(pp, threads, bytes(1), s);
+    if (dtype == DT_BF16) return group == 4 ? pick_norm_rotary<bf16, 4>(pp, threads, bytes(4), s) : pick_norm_rotary<bf16, 1>(pp, threads, bytes(1), s);
+    return fail("norm_rotary_store: unknown dtype");
 }
 
 // ---------------------------------------------------------------------------
