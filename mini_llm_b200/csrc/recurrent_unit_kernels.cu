@@ -104,11 +104,34 @@ norm_rotary_store_kernel(NormRotaryParams pp) {
             tok_place[threadIdx.x] = (long)pp.block_table[(long)item * pp.max_blocks + p / pp.page_size] * pp.page_size + (p % pp.page_size);
     }
     __syncthreads();
+    // where every token's predecessors are rows of this step, no column asks for the state (the same for all threads)
+    bool interior = TAPS > 0 && n_here == G;
+    if (TAPS > 0)
+        for (int g = 0; g < n_here; g++) interior = interior && tok_local[g] >= TAPS - 1;
 
     // column c of the block's tokens, filtered
     auto column = [&](int c, float* y) {
         const float* base = pp.qkv + c;
-        if (TAPS == 0) {
+        if (TAPS > 1 && interior) {
+            constexpr int TP = TAPS > 1 ? TAPS : 1;
+            const float* row = base + (long)(t0 - (TP - 1)) * pp.ld;
+            float u[G + TP - 1], w[TP];
+#pragma unroll
+            for (int i = 0; i < G + TP - 1; i++) u[i] = row[i * pp.ld];
+            if (TP == 4) {
+                const float4 v = *reinterpret_cast<const float4*>(pp.tap_weights + (long)c * TP);
+                w[0] = v.x, w[1 % TP] = v.y, w[2 % TP] = v.z, w[3 % TP] = v.w;
+            } else {
+#pragma unroll
+                for (int j = 0; j < TP; j++) w[j] = pp.tap_weights[(long)c * TP + j];
+            }
+#pragma unroll
+            for (int g = 0; g < G; g++) {
+                y[g] = 0.0f;
+#pragma unroll
+                for (int j = 0; j < TP; j++) y[g] = fmaf(w[j], u[g + j], y[g]);
+            }
+        } else if (TAPS == 0) {
 #pragma unroll
             for (int g = 0; g < G; g++) y[g] = g < n_here ? base[(long)(t0 + g) * pp.ld] : 0.0f;
         } else if (TAPS > 0) {

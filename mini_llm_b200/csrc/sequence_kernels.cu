@@ -111,7 +111,7 @@ extern "C" int mllm_sequence_grouped_rms_norm(void* out, long ld_out, const floa
 // if `silu` is set.  h and out may have row strides of their own (columns of a wider buffer),
 // and out may be h: a block reads its token's earlier rows, so a second buffer is needed only
 // when a step brings more than one token of a request (the launcher's caller sees to that).
-// One block per token.  A second kernel (one block per entry) then moves the state on; in a step
+// One block per token.  A second kernel (blocks per entry) then moves the state on; in a step
 // of single tokens (writes == 2) the first kernel moves it itself.
 // ---------------------------------------------------------------------------
 template <typename T>
@@ -159,7 +159,7 @@ __global__ void causal_taps_state_kernel(float* __restrict__ state, long state_s
     if (count <= 0) return;
     float* held = state + (long)item_slot[item] * state_stride;
     const long first = item_offset[item];
-    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < width; c += gridDim.y * blockDim.x) {
         // ascending: entry s takes what lay at s + count, which no earlier write has touched
         for (int s = 0; s < taps - 1; s++) {
             const int from = count - (taps - 1) + s;             // index among this step's tokens
@@ -167,6 +167,12 @@ __global__ void causal_taps_state_kernel(float* __restrict__ state, long state_s
                                                   : held[(long)(s + count) * width + c];
         }
     }
+}
+
+// An entry's channels over as many blocks as they fill (each channel is one thread's).
+static dim3 taps_state_grid(int n_items, int width) {
+    const int threads = width >= 256 ? 256 : 64;
+    return dim3(n_items, (width + threads - 1) / threads);
 }
 
 // A step of single tokens: the norm in groups, the filter and the move of its state as one kernel.
@@ -230,7 +236,7 @@ extern "C" int mllm_sequence_taps_state(float* state, long state_stride, const f
                                         const int* item_offset, const int* item_count, int n_items, int width, int taps,
                                         void* stream) {
     if (n_items <= 0 || taps <= 1) return 0;
-    launch_kernel(g_dependent_launch != 0, causal_taps_state_kernel<float>, dim3(n_items), dim3(width >= 256 ? 256 : 64), 0,
+    launch_kernel(g_dependent_launch != 0, causal_taps_state_kernel<float>, taps_state_grid(n_items, width), dim3(width >= 256 ? 256 : 64), 0,
                   (cudaStream_t)stream, state, state_stride, h, ld_h, item_slot, item_offset, item_count, width, taps);
     return check_launch("causal_taps_state_kernel");
 }
@@ -251,14 +257,14 @@ extern "C" int mllm_sequence_causal_taps(void* out, long ld_out, const void* h, 
                       (const float*)h, ld_h, w, bias, state, state_stride, positions, token_item, item_slot, item_start, width,
                       taps, identity, silu, (int)(writes == 2));
         if (writes == 1 && taps > 1)
-            launch_kernel(g_dependent_launch != 0, causal_taps_state_kernel<float>, dim3(n_items), dim3(threads), 0, s, state,
+            launch_kernel(g_dependent_launch != 0, causal_taps_state_kernel<float>, taps_state_grid(n_items, width), dim3(threads), 0, s, state,
                           state_stride, (const float*)h, ld_h, item_slot, item_offset, item_count, width, taps);
     } else if (dtype == DT_BF16) {
         launch_kernel(g_dependent_launch != 0, causal_taps_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, (bf16*)out, ld_out,
                       (const bf16*)h, ld_h, w, bias, state, state_stride, positions, token_item, item_slot, item_start, width,
                       taps, identity, silu, (int)(writes == 2));
         if (writes == 1 && taps > 1)
-            launch_kernel(g_dependent_launch != 0, causal_taps_state_kernel<bf16>, dim3(n_items), dim3(threads), 0, s, state,
+            launch_kernel(g_dependent_launch != 0, causal_taps_state_kernel<bf16>, taps_state_grid(n_items, width), dim3(threads), 0, s, state,
                           state_stride, (const bf16*)h, ld_h, item_slot, item_offset, item_count, width, taps);
     } else {
         return fail("causal_taps: unknown dtype");
