@@ -1650,7 +1650,7 @@ def nufavik_kernels(torch, size: dict, peak: dict):
             else:
                 gu = torch.empty(n, (2 if gated else 1) * total, device="cuda", dtype=torch.bfloat16)
                 act = torch.empty(n, total, device="cuda", dtype=torch.bfloat16)
-                combine = lambda i: ops.expert_combine(act, gu, choice, in_weight, out_weight, experts, inner, top, top, gated=gated,
+                combine = lambda i: ops.expert_combine(act, gu, choice, in_weight, out_weight, experts, inner, top, top, form="gated_silu" if gated else "relu_squared",
                                                        hidden=hidden, x=x, identity_weight=identity_weight)
 
                 def launch(i):

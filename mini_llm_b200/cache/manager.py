@@ -84,6 +84,8 @@ class CacheManager:
         self.max_tokens_per_request = int(max_tokens_per_request)
         self.groups: list[CacheGroup] = []
         self.entry_group: dict = {}                    # run entry, or (run entry, role) -> (group index, index within the group)
+        needs = list(needs)
+        self.n_owners = len(needs)                     # run entries, and what stands behind them (an embedding that keeps something)
         max_blocks = -(-self.max_tokens_per_request // self.page_size)
         for index, (need, entries) in enumerate(group_entries(needs)):
             group = CacheGroup(index, need, entries)

@@ -131,6 +131,10 @@ class CacheStorage:
             else:
                 self.views.append(LayerCache())
 
+        # owners behind the run entries (an embedding that keeps something per request)
+        for index in range(len(order), manager.n_owners):
+            self.views.append(view_of(index, True) if index in manager.entry_group else LayerCache())
+
         if poison is not None:
             manager.on_free = self.poison_pages
 

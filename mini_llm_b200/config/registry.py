@@ -66,4 +66,4 @@ def _load_builtin() -> None:
     global _builtin_loaded
     if not _builtin_loaded:
         _builtin_loaded = True
-        from ..models import deluvik, fuvolix, gpt2, lipulorn, nufavik, sumozen  # noqa: F401  (register themselves)
+        from ..models import deluvik, fuvolix, gpt2, kerepel, lipulorn, nufavik, sumozen  # noqa: F401  (register themselves)

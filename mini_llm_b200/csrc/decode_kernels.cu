@@ -234,7 +234,7 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
                        const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                        const int* __restrict__ token_item, int n_heads, int n_kv_heads, int dim, int vdim, int page_size,
                        float scale, float cap, int window, int block, int keep, const float* __restrict__ gate, long ld_gate,
-                       const float* __restrict__ sink, int chunk, int max_chunks, float* __restrict__ part_acc,
+                       int gate_wide, const float* __restrict__ sink, const float* __restrict__ slopes, int chunk, int max_chunks, float* __restrict__ part_acc,
                        float* __restrict__ part_ml, int* __restrict__ counters) {
     if (FULL) dim = vdim = D;
     constexpr int LPK = D / 8;             // lanes per key: each lane owns 8 of the head's dimensions
@@ -266,6 +266,8 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
     const float scale_log2 = scale * 1.4426950408889634f;
     // a cap on the scores, cap * tanh(score / cap), in the same units (cap <= 0: none)
     const float cap_log2 = cap * 1.4426950408889634f, inv_cap_log2 = cap > 0.0f ? 1.0f / cap_log2 : 0.0f;
+    // a bias by distance, taken off the (capped) score, in the same units
+    const float slope_log2 = slopes != nullptr ? slopes[h] * 1.4426950408889634f : 0.0f;
 #pragma unroll
     for (int i = 0; i < 8; i++) {
         qf[i] *= scale_log2;
@@ -309,7 +311,8 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
         float sc[2], vf[2][8];
 #pragma unroll
         for (int u = 0; u < 2; u++) {
-            const bool valid = first_key + trip * 8 * KPW + u * 4 * KPW <= end;
+            const int number = first_key + trip * 8 * KPW + u * 4 * KPW;
+            const bool valid = number <= end;
             float kf[8];
             unpack8(has_key ? ring[trip % RING][u][0][threadIdx.x] : make_uint4(0u, 0u, 0u, 0u), kf);
             unpack8(has_value ? ring[trip % RING][u][1][threadIdx.x] : make_uint4(0u, 0u, 0u, 0u), vf[u]);
@@ -319,6 +322,7 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
 #pragma unroll
             for (int o = LPK / 2; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
             if (cap > 0.0f) dot = cap_log2 * tanhf(dot * inv_cap_log2);
+            dot = fmaf(-slope_log2, (float)(p - (number < n_kept ? number : number + gap)), dot);
             sc[u] = valid ? dot : -INFINITY;          // what an absent key left in the ring is never used
             if (!valid) {
 #pragma unroll
@@ -392,9 +396,9 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
     float denom = sink != nullptr ? exp2f(sink_log2 - top) : 0.0f;
     for (int cc = 0; cc <= c_last; cc++)
         denom += __ldcg(part_ml + (first + cc) * 2 + 1) * exp2f(__ldcg(part_ml + (first + cc) * 2) - top);
-    // a gate per (token, head) opens the result by its sigmoid
-    const float open = gate != nullptr ? 1.0f / (1.0f + __expf(-gate[(long)t * ld_gate + h])) : 1.0f;
     for (int d = threadIdx.x; d < vdim; d += 128) {
+        // a gate per (token, head), or per entry of the head's result, opens it by its sigmoid
+        const float open = gate != nullptr ? 1.0f / (1.0f + __expf(-gate[(long)t * ld_gate + (gate_wide ? h * vdim + d : h)])) : 1.0f;
         float o = 0.0f;
         for (int cc = 0; cc <= c_last; cc++)
             o += __ldcg(part_acc + (first + cc) * D + d) * exp2f(__ldcg(part_ml + (first + cc) * 2) - top);
@@ -404,7 +408,8 @@ split_attention_kernel(bf16* __restrict__ out, long ld_out, const bf16* __restri
 
 // (with a cap on the scores: score <- cap * tanh(score / cap); cap <= 0: none; with a mask of blocks of
 // positions: block > 0, a query sees only keys of its own block, counted from position 0; with a gate:
-// fp32 [tokens, >= heads], head h's result times sigmoid(gate[t, h]); with a sink: fp32 [heads], exp(sink[h]) joins
+// fp32 [tokens, >= heads], head h's result times sigmoid(gate[t, h]), or with gate_wide [tokens, >= heads * vdim], entry d
+// of it times sigmoid(gate[t, h * vdim + d]); with slopes: fp32 [heads], slopes[h] * (distance) comes off the score; with a sink: fp32 [heads], exp(sink[h]) joins
 // head h's softmax denominator)
 // The widest form: key rows of `dim` and value rows of `vdim` entries (equal and one of 16, 32, 64, 128, 256, or
 // any multiples of 8 up to 256; the scratch's rows then have the least of those sizes that holds both), and the keys
@@ -414,7 +419,7 @@ extern "C" int mllm_decode_split_attention_kept(void* out, long ld_out, const vo
                                                 const int* positions, const int* token_item, int n_tokens, int n_heads,
                                                 int n_kv_heads, int dim, int vdim, int page_size, float scale, float cap,
                                                 int window, int block, int keep, const float* gate, long ld_gate,
-                                                const float* sink, int chunk, int max_chunks, float* part_acc,
+                                                int gate_wide, const float* sink, const float* slopes, int chunk, int max_chunks, float* part_acc,
                                                 float* part_ml, int* counters, void* stream) {
     if (n_tokens <= 0) return 0;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0)
@@ -434,7 +439,7 @@ extern "C" int mllm_decode_split_attention_kept(void* out, long ld_out, const vo
     launch_kernel(g_dependent_launch != 0, split_attention_kernel<D, FULL>, grid, dim3(128), 0, s, (bf16*)out, ld_out, \
                   (const bf16*)q, ld_q, (const bf16*)k_pages, (const bf16*)v_pages, block_table, max_blocks,         \
                   positions, token_item, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, block, keep, \
-                  gate, ld_gate, sink, chunk, max_chunks, part_acc, part_ml, counters)
+                  gate, ld_gate, gate_wide, sink, slopes, chunk, max_chunks, part_acc, part_ml, counters)
 #define PICK_SPLIT(D) do { if (full) LAUNCH_SPLIT(D, true); else LAUNCH_SPLIT(D, false); } while (0)
     switch (size) {
     case 16: PICK_SPLIT(16); break;
@@ -461,8 +466,8 @@ extern "C" int mllm_decode_split_attention_sink(void* out, long ld_out, const vo
     }
     return mllm_decode_split_attention_kept(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions,
                                             token_item, n_tokens, n_heads, n_kv_heads, head_size, head_size, page_size, scale,
-                                            cap, window, block, 0, gate, ld_gate, sink, chunk, max_chunks, part_acc, part_ml,
-                                            counters, stream);
+                                            cap, window, block, 0, gate, ld_gate, 0, sink, nullptr, chunk, max_chunks, part_acc,
+                                            part_ml, counters, stream);
 }
 
 extern "C" int mllm_decode_split_attention_masked(void* out, long ld_out, const void* q, long ld_q, const void* k_pages,

@@ -165,7 +165,9 @@ extern "C" int mllm_hybrid_head_norm_store(void* qkv, long ld, int k_off, int v_
 // ---------------------------------------------------------------------------
 // Causal attention with capped scores, one block per (token, head): the plain form, which takes
 // every size.  score = cap * tanh((q . k) * scale / cap) (cap <= 0: no cap); the query at position
-// p sees keys max(0, p - window + 1) .. p (window <= 0: all) and those below `keep`.  Four warps take the keys in turn,
+// p sees keys max(0, p - window + 1) .. p (window <= 0: all) and those below `keep`.  With `slopes` [heads] a bias
+// by distance comes off the (capped) score: slopes[h] * (p - j) for key j.  `gate` opens the result by a sigmoid: one number per head
+// (gate[t, h]) or, with gate_wide, one per entry (gate[t, h * vdim + d]).  Four warps take the keys in turn,
 // each with an online softmax; their states are merged in a fixed order.
 // ---------------------------------------------------------------------------
 constexpr int CAP_MAX_HEAD = 256;
@@ -196,7 +198,8 @@ capped_attention_plain_kernel(T* __restrict__ out, long ld_out, const T* __restr
                               const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                               const int* __restrict__ token_item, int n_heads, int n_kv_heads, int dim, int vdim,
                               int page_size, float scale, float cap, int window, int chunk, int keep,
-                              const float* __restrict__ gate, long ld_gate, const float* __restrict__ sink) {
+                              const float* __restrict__ gate, long ld_gate, int gate_wide, const float* __restrict__ sink,
+                              const float* __restrict__ slopes) {
     dependents_may_start();
     wait_for_earlier_kernels();
     constexpr int R = CAP_MAX_HEAD / 32;
@@ -214,6 +217,7 @@ capped_attention_plain_kernel(T* __restrict__ out, long ld_out, const T* __restr
         acc[i] = 0.0f;
     }
     float m = -INFINITY, l = 0.0f;
+    const float slope = slopes != nullptr ? slopes[h] : 0.0f;
     const int lo = first_visible(p, window, chunk);
     const int n_kept = min(keep, lo);                        // kept keys ahead of the window, then the window's
     for (int i = warp; i <= p - lo + n_kept; i += 4) {
@@ -227,7 +231,7 @@ capped_attention_plain_kernel(T* __restrict__ out, long ld_out, const T* __restr
             const int d = lane + 32 * i;
             if (d < dim) s = fmaf(qr[i], to_f32(kr[d]), s);
         }
-        s = capped(warp_sum(s) * scale, cap, inv_cap);
+        s = capped(warp_sum(s) * scale, cap, inv_cap) - slope * (float)(p - j);
         const float m_new = fmaxf(m, s);
         const float c = expf(m - m_new), e = expf(s - m_new);
         l = l * c + e;
@@ -256,8 +260,8 @@ capped_attention_plain_kernel(T* __restrict__ out, long ld_out, const T* __restr
         wgt[w] = sm_m[w] == -INFINITY ? 0.0f : expf(sm_m[w] - big);
         total += sm_l[w] * wgt[w];
     }
-    const float open = gate != nullptr ? sigmoid_f(gate[(long)t * ld_gate + h]) : 1.0f;
     for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
+        const float open = gate != nullptr ? sigmoid_f(gate[(long)t * ld_gate + (gate_wide ? h * vdim + d : h)]) : 1.0f;
         float o = 0.0f;
 #pragma unroll
         for (int w = 0; w < 4; w++) o += sm_acc[w][d] * wgt[w];
@@ -299,8 +303,8 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
                               const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                               const int* __restrict__ token_item, int n_tokens, int n_heads, int n_kv_heads, int dim,
                               int vdim, int page_size, float scale, float cap, int window, int chunk, int keep,
-                              const float* __restrict__ gate, long ld_gate, const float* __restrict__ sink,
-                              int tokens_per_block, int heads_per_block) {
+                              const float* __restrict__ gate, long ld_gate, int gate_wide, const float* __restrict__ sink,
+                              const float* __restrict__ slopes, int tokens_per_block, int heads_per_block) {
     dependents_may_start();
     wait_for_earlier_kernels();
     constexpr int ROWS = TILE_WARPS * R;
@@ -324,7 +328,7 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
 
     // this warp's rows: r = warp + s * TILE_WARPS; row r = (token r / heads, head r % heads)
     int row_pos[R], row_item[R];
-    float m[R], l[R], acc[R][VPL];
+    float m[R], l[R], acc[R][VPL], slope[R];
 #pragma unroll
     for (int s = 0; s < R; s++) {
         const int r = warp + s * TILE_WARPS;
@@ -332,6 +336,7 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
         const int token = live ? first_token + r / n_heads_here : 0;
         row_pos[s] = live ? positions[token] : -1;
         row_item[s] = live ? token_item[token] : -1;
+        slope[s] = live && slopes != nullptr ? slopes[first_head + r % n_heads_here] : 0.0f;
         m[s] = -INFINITY, l[s] = 0.0f;
 #pragma unroll
         for (int i = 0; i < VPL; i++) acc[s][i] = 0.0f;
@@ -430,7 +435,7 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
 #pragma unroll
             for (int s = 0; s < R; s++) {
                 const bool mine = seen[s] && lane < n_keys && pos <= row_pos[s] && key_visible(pos, first_seen[s], keep);
-                const float score = mine ? capped(dot[s] * scale, cap, inv_cap) : -INFINITY;
+                const float score = mine ? capped(dot[s] * scale, cap, inv_cap) - slope[s] * (float)(row_pos[s] - pos) : -INFINITY;
                 const float block_max = warp_max(score);
                 float rescale = 1.0f, e = 0.0f;
                 if (block_max != -INFINITY) {
@@ -480,17 +485,19 @@ capped_attention_tiled_kernel(T* __restrict__ out, long ld_out, const T* __restr
             shrink = expf(m[s] - top);
             sum = sum * shrink + expf(sink[head] - top);
         }
-        const float inv = (gate != nullptr ? sigmoid_f(gate[(long)token * ld_gate + head]) : 1.0f) * shrink / sum;
+        const float inv = (gate != nullptr && !gate_wide ? sigmoid_f(gate[(long)token * ld_gate + head]) : 1.0f) * shrink / sum;
 #pragma unroll
         for (int i = 0; i < VPL; i++) {
             const int d = lane + 32 * i;
-            if (d < vdim) out[(long)token * ld_out + (long)head * vdim + d] = from_f32<T>(acc[s][i] * inv);
+            if (d >= vdim) continue;
+            const float open = gate != nullptr && gate_wide ? sigmoid_f(gate[(long)token * ld_gate + (long)head * vdim + d]) : 1.0f;
+            out[(long)token * ld_out + (long)head * vdim + d] = from_f32<T>(acc[s][i] * inv * open);
         }
     }
 }
 
 // ---------------------------------------------------------------------------
-// The same attention as register tiles, for the common sizes (keys and values of up to 128 entries, no gate, no
+// The same attention as register tiles, for the common sizes (keys and values of up to 128 entries, no
 // mask of blocks).  A block of 256 threads takes 64 (token, head) rows of one key/value head and walks
 // the keys 64 at a time.  Thread (ty, tx) of a 16 x 16 grid holds the scores of rows 4 ty .. 4 ty + 3 against keys
 // tx, tx + 16, tx + 32, tx + 48 (sixteen sums, fed by 16-byte reads of q and k rows along the head: eight FMAs a
@@ -511,7 +518,8 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
                               const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                               const int* __restrict__ token_item, int n_tokens, int n_heads, int n_kv_heads, int dim,
                               int vdim, int page_size, float scale, float cap, int window, int keep,
-                              const float* __restrict__ sink, int tokens_per_block, int heads_per_block) {
+                              const float* __restrict__ gate, long ld_gate, int gate_wide, const float* __restrict__ sink,
+                              const float* __restrict__ slopes, int tokens_per_block, int heads_per_block) {
     dependents_may_start();
     wait_for_earlier_kernels();
     constexpr int VDIM = 64 * VG;
@@ -553,9 +561,11 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
     __syncthreads();
     constexpr int RT = BLOCK_RT;
     int my_pos[RT], my_item[RT], my_first[RT];
-    float m[RT], l[RT], o[RT][4 * VG];
+    float m[RT], l[RT], o[RT][4 * VG], slope[RT];
 #pragma unroll
     for (int i = 0; i < RT; i++) {
+        const int r = ty * RT + i;
+        slope[i] = slopes != nullptr && r < n_rows ? slopes[first_head + r % n_heads_here] : 0.0f;
         my_pos[i] = row_pos[ty * RT + i], my_item[i] = row_item[ty * RT + i];
         my_first[i] = first_visible(my_pos[i], window, 0);
         m[i] = -INFINITY, l[i] = 0.0f;
@@ -663,7 +673,7 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
                 for (int j = 0; j < 4; j++) {
                     const int pos = base + tx + 16 * j;
                     const bool seen = row_here && pos <= my_pos[i] && key_visible(pos, my_first[i], keep);
-                    score[j] = seen ? capped(acc[i][j] * scale, cap, inv_cap) : -INFINITY;
+                    score[j] = seen ? capped(acc[i][j] * scale, cap, inv_cap) - slope[i] * (float)(my_pos[i] - pos) : -INFINITY;
                     top = fmaxf(top, score[j]);
                 }
 #pragma unroll
@@ -724,13 +734,17 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
             shrink = expf(m[i] - top);
             sum = sum * shrink + expf(sink[head] - top);
         }
-        const float inv = shrink / sum;
+        const float inv = (gate != nullptr && !gate_wide ? sigmoid_f(gate[(long)token * ld_gate + head]) : 1.0f) * shrink / sum;
+        const float* open = gate != nullptr && gate_wide ? gate + (long)token * ld_gate + (long)head * vdim : nullptr;
 #pragma unroll
         for (int g = 0; g < VG; g++)
 #pragma unroll
-            for (int c = 0; c < 4; c++)
-                if (64 * g + tx * 4 + c < vdim)
-                    out[(long)token * ld_out + (long)head * vdim + 64 * g + tx * 4 + c] = from_f32<T>(o[i][4 * g + c] * inv);
+            for (int c = 0; c < 4; c++) {
+                const int d = 64 * g + tx * 4 + c;
+                if (d < vdim)
+                    out[(long)token * ld_out + (long)head * vdim + d] =
+                        from_f32<T>(o[i][4 * g + c] * inv * (open != nullptr ? sigmoid_f(open[d]) : 1.0f));
+            }
     }
 }
 
@@ -748,7 +762,8 @@ template <typename T, int VG>
 static int launch_capped_block(void* out, long ld_out, const void* q, long ld_q, const void* k_pages, const void* v_pages,
                                const int* block_table, int max_blocks, const int* positions, const int* token_item, int n_tokens,
                                int n_heads, int n_kv_heads, int dim, int vdim, int page_size, float scale, float cap, int window,
-                               int keep, const float* sink, cudaStream_t s) {
+                               int keep, const float* gate, long ld_gate, int gate_wide, const float* sink, const float* slopes,
+                               cudaStream_t s) {
     const int group = n_heads / n_kv_heads;
     const int heads_per_block = group < BLOCK_ROWS ? group : BLOCK_ROWS;
     const int tokens_per_block = BLOCK_ROWS / heads_per_block;
@@ -760,7 +775,8 @@ static int launch_capped_block(void* out, long ld_out, const void* q, long ld_q,
     dim3 grid((n_tokens + tokens_per_block - 1) / tokens_per_block, n_kv_heads * chunks);
     launch_kernel(g_dependent_launch != 0, capped_attention_block_kernel<T, VG>, grid, dim3(BLOCK_THREADS), shared, s, (T*)out, ld_out, (const T*)q,
                   ld_q, (const T*)k_pages, (const T*)v_pages, block_table, max_blocks, positions, token_item, n_tokens, n_heads,
-                  n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, sink, tokens_per_block, heads_per_block);
+                  n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, gate, ld_gate, gate_wide, sink, slopes,
+                  tokens_per_block, heads_per_block);
     return check_launch("capped_attention_block_kernel");
 }
 
@@ -779,7 +795,8 @@ template <typename T, int R, int SIZE>
 static int launch_capped_tiles(void* out, long ld_out, const void* q, long ld_q, const void* k_pages, const void* v_pages,
                                const int* block_table, int max_blocks, const int* positions, const int* token_item, int n_tokens,
                                int n_heads, int n_kv_heads, int dim, int vdim, int page_size, float scale, float cap, int window,
-                               int chunk, int keep, const float* gate, long ld_gate, const float* sink, cudaStream_t s) {
+                               int chunk, int keep, const float* gate, long ld_gate, int gate_wide, const float* sink,
+                               const float* slopes, cudaStream_t s) {
     constexpr int ROWS = TILE_WARPS * R;
     const int group = n_heads / n_kv_heads;
     const int heads_per_block = group < ROWS ? group : ROWS;
@@ -793,8 +810,8 @@ static int launch_capped_tiles(void* out, long ld_out, const void* q, long ld_q,
     dim3 grid((n_tokens + tokens_per_block - 1) / tokens_per_block, n_kv_heads * chunks);
     launch_kernel(g_dependent_launch != 0, capped_attention_tiled_kernel<T, R, SIZE>, grid, dim3(TILE_WARPS * 32), shared, s, (T*)out,
                   ld_out, (const T*)q, ld_q, (const T*)k_pages, (const T*)v_pages, block_table, max_blocks, positions, token_item,
-                  n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, sink,
-                  tokens_per_block, heads_per_block);
+                  n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, gate_wide, sink,
+                  slopes, tokens_per_block, heads_per_block);
     return check_launch("capped_attention_tiled_kernel");
 }
 
@@ -803,21 +820,24 @@ static int launch_capped_attention(bool tiled, void* out, long ld_out, const voi
                                    const void* v_pages, const int* block_table, int max_blocks, const int* positions,
                                    const int* token_item, int n_tokens, int n_heads, int n_kv_heads, int dim, int vdim,
                                    int page_size, float scale, float cap, int window, int chunk, int keep, const float* gate,
-                                   long ld_gate, const float* sink, cudaStream_t s) {
+                                   long ld_gate, int gate_wide, const float* sink, const float* slopes, cudaStream_t s) {
     if (!tiled) {
         launch_kernel(g_dependent_launch != 0, capped_attention_plain_kernel<T>, dim3(n_tokens, n_heads), dim3(128), 0, s, (T*)out,
                       ld_out, (const T*)q, ld_q, (const T*)k_pages, (const T*)v_pages, block_table, max_blocks, positions,
-                      token_item, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, sink);
+                      token_item, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, gate_wide,
+                      sink, slopes);
         return check_launch("capped_attention_plain_kernel");
     }
     // the common sizes go to the register tiles
-    if (gate == nullptr && chunk == 0 && n_tokens * (long)n_heads >= 2048 && capped_block_takes(dim, vdim, 16 / (int)sizeof(T)) &&
+    if (chunk == 0 && n_tokens * (long)n_heads >= 2048 && capped_block_takes(dim, vdim, 16 / (int)sizeof(T)) &&
         (ld_q * sizeof(T)) % 16 == 0) {
         if (vdim <= 64)
             return launch_capped_block<T, 1>(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions, token_item,
-                                             n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, sink, s);
+                                             n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, gate, ld_gate,
+                                             gate_wide, sink, slopes, s);
         return launch_capped_block<T, 2>(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions, token_item,
-                                         n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, sink, s);
+                                         n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, keep, gate, ld_gate,
+                                             gate_wide, sink, slopes, s);
     }
     // rows a warp: four where the step has rows enough for the blocks to fill the GPU all the same
     // (and their shared memory fits), else two
@@ -826,7 +846,8 @@ static int launch_capped_attention(bool tiled, void* out, long ld_out, const voi
     if (capped_tiled_shared(dim, vdim, per_warp) > 160 * 1024) per_warp = 2;
 #define TILES(R, SIZE)                                                                                                        \
     return launch_capped_tiles<T, R, SIZE>(out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions, token_item, \
-                                           n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, sink, s)
+                                           n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep, gate, ld_gate, gate_wide, \
+                                           sink, slopes, s)
     const int size = (dim > vdim ? dim : vdim) <= 64 ? 64 : ((dim > vdim ? dim : vdim) <= 128 ? 128 : 256);
     if (per_warp == 4) { if (size == 64) TILES(4, 64); if (size == 128) TILES(4, 128); TILES(4, 256); }
     if (size == 64) TILES(2, 64);
@@ -839,7 +860,8 @@ extern "C" int mllm_hybrid_capped_attention(void* out, long ld_out, const void* 
                                             const void* v_pages, const int* block_table, int max_blocks, const int* positions,
                                             const int* token_item, int n_tokens, int n_heads, int n_kv_heads, int dim, int vdim,
                                             int page_size, float scale, float cap, int window, int chunk, int keep, const float* gate,
-                                            long ld_gate, const float* sink, int tiled, int dtype, void* stream) {
+                                            long ld_gate, int gate_wide, const float* sink, const float* slopes, int tiled, int dtype,
+                                            void* stream) {
     if (n_tokens <= 0) return 0;
     if (dim <= 0 || dim > CAP_MAX_HEAD || vdim <= 0 || vdim > CAP_MAX_HEAD) return fail("capped_attention: key and value sizes must be in 1..256");
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0) return fail("capped_attention: heads must be a multiple of the key/value heads");
@@ -850,11 +872,11 @@ extern "C" int mllm_hybrid_capped_attention(void* out, long ld_out, const void* 
     if (dtype == DT_F32)
         return launch_capped_attention<float>(tiled != 0, out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions,
                                               token_item, n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep,
-                                              gate, ld_gate, sink, s);
+                                              gate, ld_gate, gate_wide, sink, slopes, s);
     if (dtype == DT_BF16)
         return launch_capped_attention<bf16>(tiled != 0, out, ld_out, q, ld_q, k_pages, v_pages, block_table, max_blocks, positions,
                                              token_item, n_tokens, n_heads, n_kv_heads, dim, vdim, page_size, scale, cap, window, chunk, keep,
-                                             gate, ld_gate, sink, s);
+                                             gate, ld_gate, gate_wide, sink, slopes, s);
     return fail("capped_attention: unknown dtype");
 }
 
@@ -1198,10 +1220,15 @@ extern "C" int mllm_hybrid_linear_recurrence(const RecurrenceParams* params, int
 //                chosen ones' OUTPUTS are weighed by the softmax over the chosen logits only, and
 //                their inputs by 1.  ROUTE_SOFTMAX_OF_ALL: s = the softmax over all outputs; s plus a
 //                correction per output ranks them, the chosen ones' outputs are weighed by s over
-//                the chosen ones' sum (+ 1e-20), times `scale`.  The last `n_identity` outputs are
+//                the chosen ones' sum (+ 1e-20), times `scale`.  ROUTE_SIGMOID: s = sigmoid(z); s plus a
+//                correction ranks, the chosen ones' outputs are weighed by s itself, times `scale`.  With
+//                `groups` the experts form that many equal runs of neighbours, of which only the `keep`
+//                best can be chosen from; a group's score is the sum of its two largest ranking scores.
+//                The last `n_identity` outputs are
 //                identity experts, whose output is the token itself: such a choice becomes -1 and
 //                its weight goes into the token's identity weight
-//   expert_up    act[pair, f] = silu(W_gate[e] x') * (W_up[e] x') with x' = weight * x
+//   expert_up    act[pair, f] = silu(W_gate[e] x') * (W_up[e] x') with x' = weight * x (or another form of
+//                an expert, see ExpertForm)
 //   expert_down  hidden[t] += sum over the token's pairs of out_weight * W_down[e] act[pair] (or, with `assign`,
 //                hidden[t] = that sum)
 // Experts are named by a table of pointers (gate, up, down) and inner sizes, so that experts of
@@ -1238,7 +1265,7 @@ __device__ __forceinline__ bool aligned16(const void* p) { return (reinterpret_c
 static bool aligned_host(const void* p) { return (reinterpret_cast<unsigned long long>(p) & 15ull) == 0; }
 
 // How a token's experts are chosen and weighed (the launcher's `rule`).
-enum RouteRule { ROUTE_SIGMOID_ON_INPUT = 0, ROUTE_SOFTMAX_OF_CHOSEN = 1, ROUTE_SOFTMAX_OF_ALL = 2 };
+enum RouteRule { ROUTE_SIGMOID_ON_INPUT = 0, ROUTE_SOFTMAX_OF_CHOSEN = 1, ROUTE_SOFTMAX_OF_ALL = 2, ROUTE_SIGMOID = 3 };
 
 // A block takes TOKENS consecutive tokens (four in long steps: a router row that is read serves all of them) and deals
 // the outputs out to its warps; then a warp a token ranks.
@@ -1246,14 +1273,15 @@ template <typename T, int TOKENS>
 __global__ void __launch_bounds__(512)
 route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, const float* __restrict__ router_bias,
              const float* __restrict__ correction, const T* __restrict__ shared_gate, int shared_plain, int rule, float scale,
-             int width, int n_outputs, int n_identity, int top, int pairs, int n_tokens, int* __restrict__ choice,
-             float* __restrict__ in_weight, float* __restrict__ out_weight, float* __restrict__ identity_weight) {
+             int width, int n_outputs, int n_identity, int groups, int keep_groups, int top, int pairs, int n_tokens,
+             int* __restrict__ choice, float* __restrict__ in_weight, float* __restrict__ out_weight, float* __restrict__ identity_weight) {
     dependents_may_start();
     wait_for_earlier_kernels();
     extern __shared__ __align__(16) float shared[];
     float* rows = shared;                                  // [TOKENS][width]
     float* scores = rows + TOKENS * width;                 // [TOKENS][n_outputs + 1]: what ranks the experts
-    float* shares = scores + TOKENS * (n_outputs + 1);     // [TOKENS][n_outputs]: the softmax over all outputs (ROUTE_SOFTMAX_OF_ALL)
+    float* shares = scores + TOKENS * (n_outputs + 1);     // [TOKENS][n_outputs]: what weighs them where that is something else
+    float* group_scores = shares + TOKENS * n_outputs;     // [TOKENS][groups]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
     const int t0 = blockIdx.x * TOKENS, n_here = min(TOKENS, n_tokens - t0);
     constexpr int N = Vec16<T>::N;
@@ -1297,7 +1325,8 @@ route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, c
             float sum = warp_sum(z[g]);
             if (e < n_outputs && router_bias != nullptr) sum += router_bias[e];
             // (a softmax needs the logits themselves)
-            if (lane == 0) scores[g * (n_outputs + 1) + e] = rule != ROUTE_SIGMOID_ON_INPUT && e < n_outputs ? sum : sigmoid_f(sum);
+            const bool logit = (rule == ROUTE_SOFTMAX_OF_CHOSEN || rule == ROUTE_SOFTMAX_OF_ALL) && e < n_outputs;
+            if (lane == 0) scores[g * (n_outputs + 1) + e] = logit ? sum : sigmoid_f(sum);
         }
     }
     __syncthreads();
@@ -1320,6 +1349,36 @@ route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, c
         }
         __syncwarp();
     }
+    if (rule == ROUTE_SIGMOID) {
+        for (int e = lane; e < n_outputs; e += 32) {
+            share[e] = score[e];
+            score[e] += correction != nullptr ? correction[e] : 0.0f;
+        }
+        __syncwarp();
+    }
+    if (groups > 0) {
+        // a lane sums its groups' two best; then the groups that keep_groups others beat (the lower index wins a tie) drop out
+        float* group_score = group_scores + warp * groups;
+        const int size = n_outputs / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float first = -INFINITY, second = -INFINITY;
+            for (int e = g * size; e < (g + 1) * size; e++) {
+                const float v = score[e];
+                if (v > first) second = first, first = v;
+                else if (v > second) second = v;
+            }
+            group_score[g] = size > 1 ? first + second : first;
+        }
+        __syncwarp();
+        for (int e = lane; e < n_outputs; e += 32) {
+            const int mine = e / size;
+            int ahead = 0;
+            for (int g = 0; g < groups; g++)
+                ahead += group_score[g] > group_score[mine] || (group_score[g] == group_score[mine] && g < mine) ? 1 : 0;
+            if (ahead >= keep_groups) score[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     const int n_real = n_outputs - n_identity;
     float largest = 0.0f, total = 0.0f;
     for (int k = 0; k < top; k++) {
@@ -1337,7 +1396,7 @@ route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, c
         if (k == 0) largest = best_score;                            // (the first is the largest)
         float weight = best_score;
         if (rule == ROUTE_SOFTMAX_OF_CHOSEN) weight = expf(best_score - largest);
-        if (rule == ROUTE_SOFTMAX_OF_ALL) weight = share[best];
+        if (rule == ROUTE_SOFTMAX_OF_ALL || rule == ROUTE_SIGMOID) weight = share[best];
         total += weight;
         if (lane == 0) {
             const long pair = (long)t * pairs + k;
@@ -1354,7 +1413,8 @@ route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, c
         float passed = 0.0f;
         for (int k = 0; k < top; k++) {
             const long pair = (long)t * pairs + k;
-            const float weight = rule == ROUTE_SOFTMAX_OF_ALL ? out_weight[pair] / (total + 1e-20f) * scale : out_weight[pair] / total;
+            const float over = rule == ROUTE_SIGMOID ? 1.0f : (rule == ROUTE_SOFTMAX_OF_ALL ? total + 1e-20f : total);
+            const float weight = out_weight[pair] / over * (rule == ROUTE_SOFTMAX_OF_CHOSEN ? 1.0f : scale);
             const bool identity = choice[pair] >= n_real;
             if (identity) passed += weight, choice[pair] = -1;
             out_weight[pair] = identity ? 0.0f : weight;
@@ -1368,18 +1428,31 @@ route_kernel(const T* __restrict__ x, long ld_x, const T* __restrict__ router, c
     }
 }
 
-// What an expert applies between its two products: silu(gate) * up, or (no gate matrix) the square of relu(up).
-__device__ __forceinline__ float relu_squared(float z) {
-    const float r = fmaxf(z, 0.0f);
-    return r * r;
+// What an expert applies between its two products: silu(gate) * up; (no gate matrix) the square of relu(up); or, with
+// both products clamped, g' * sigmoid(alpha g') * (u' + 1) for g' = min(gate, limit), u' = clamp(up, -limit, limit).
+enum ExpertForm { EXPERT_GATED_SILU = 0, EXPERT_RELU_SQUARED = 1, EXPERT_CLAMPED_GLU = 2 };
+
+template <int FORM> __device__ __forceinline__ float expert_form(float g, float u, float limit, float alpha) {
+    if (FORM == EXPERT_RELU_SQUARED) {
+        const float r = fmaxf(u, 0.0f);
+        return r * r;
+    }
+    if (FORM == EXPERT_CLAMPED_GLU) {
+        g = fminf(g, limit), u = fminf(fmaxf(u, -limit), limit);
+        return g * sigmoid_f(alpha * g) * (u + 1.0f);
+    }
+    return silu_f(g) * u;
 }
 
 // A warp takes F inner features of a pair at once: their rows' loads do not wait on one another.
-template <typename T, bool GATED, int F>
+// (the routed experts share one limit; expert `n_experts`, the shared one, has its own)
+template <typename T, int FORM, int F>
 __global__ void __launch_bounds__(256)
 expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long ld_x, const int* __restrict__ choice,
                  const float* __restrict__ in_weight, const long long* __restrict__ gate_of, const long long* __restrict__ up_of,
-                 const int* __restrict__ inner_of, int width, int pairs) {
+                 const int* __restrict__ inner_of, int width, int pairs, float limit, float shared_limit, float alpha,
+                 int n_experts) {
+    constexpr bool GATED = FORM != EXPERT_RELU_SQUARED;
     dependents_may_start();
     wait_for_earlier_kernels();
     extern __shared__ __align__(16) float row[];             // [width]: the token times its weight, rounded as an activation
@@ -1435,7 +1508,8 @@ expert_up_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ x, long
 #pragma unroll
     for (int k = 0; k < F; k++) {
         const float g = GATED ? warp_sum(zg[k]) : 0.0f, u = warp_sum(zu[k]);
-        if (lane == 0 && f0 + k < inner) act[(long)pair * ld_act + f0 + k] = from_f32<T>(GATED ? silu_f(g) * u : relu_squared(u));
+        if (lane == 0 && f0 + k < inner)
+            act[(long)pair * ld_act + f0 + k] = from_f32<T>(expert_form<FORM>(g, u, e == n_experts ? shared_limit : limit, alpha));
     }
 }
 
@@ -1507,15 +1581,17 @@ expert_down_kernel(float* __restrict__ hidden, long ld_hidden, const T* __restri
 // (VEC: a thread takes the 16 bytes of columns that lie side by side, all of one expert: inner sizes that are
 // multiples of a vector's elements.  The token's weights per expert lie in shared memory, 0 for an expert it
 // did not choose, whose columns are written as zeros without reading the products.)
-// (GATED false: experts without a gate matrix; gu holds the ups alone, [T, total], and act is the square of relu.
+// (EXPERT_RELU_SQUARED: experts without a gate matrix; gu holds the ups alone, [T, total], and act is the square of relu.
 // With `identity_weight` the block's share of the token's columns of `hidden` also gets identity_weight[t] * x[t]:
 // set to it with `assign`, else added.)
-template <typename T, bool VEC, bool GATED>
+template <typename T, bool VEC, int FORM>
 __global__ void __launch_bounds__(256)
 expert_combine_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ gu, long ld_gu, const int* __restrict__ choice,
                       const float* __restrict__ in_weight, const float* __restrict__ out_weight, int n_experts, int inner,
                       int total, int top, int pairs, float* __restrict__ hidden, long ld_hidden, const T* __restrict__ x,
-                      long ld_x, const float* __restrict__ identity_weight, int width, int assign) {
+                      long ld_x, const float* __restrict__ identity_weight, int width, int assign, float limit,
+                      float shared_limit, float alpha) {
+    constexpr bool GATED = FORM != EXPERT_RELU_SQUARED;
     dependents_may_start();
     wait_for_earlier_kernels();
     extern __shared__ float weights[];             // [n_experts + 1][2]: input weight, output weight
@@ -1537,22 +1613,23 @@ expert_combine_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ gu
     for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * N; c < total; c += gridDim.y * blockDim.x * N) {
         const int e = c < n_experts * inner ? c / inner : n_experts;
         const float s = weights[2 * e], o = weights[2 * e + 1];
+        const float most = e == n_experts ? shared_limit : limit;
         if (VEC) {
             uint4 packed = make_uint4(0u, 0u, 0u, 0u);
             if (s != 0.0f) {
                 float g[N], u[N];
-                Vec16<T>::load(row + c, g);
-                if (GATED) Vec16<T>::load(row + total + c, u);
+                if (GATED) Vec16<T>::load(row + c, g);
+                Vec16<T>::load(row + (GATED ? total : 0) + c, u);
                 T* lanes = reinterpret_cast<T*>(&packed);
 #pragma unroll
                 for (int i = 0; i < N; i++)
-                    lanes[i] = from_f32<T>(GATED ? silu_f(s * g[i]) * (s * u[i]) * o : relu_squared(s * g[i]) * o);
+                    lanes[i] = from_f32<T>(expert_form<FORM>(GATED ? s * g[i] : 0.0f, s * u[i], most, alpha) * o);
             }
             *reinterpret_cast<uint4*>(dst + c) = packed;
         } else {
             float v = 0.0f;
-            if (s != 0.0f && GATED) v = silu_f(s * to_f32(row[c])) * (s * to_f32(row[total + c])) * o;
-            if (s != 0.0f && !GATED) v = relu_squared(s * to_f32(row[c])) * o;
+            if (s != 0.0f)
+                v = expert_form<FORM>(GATED ? s * to_f32(row[c]) : 0.0f, s * to_f32(row[(GATED ? total : 0) + c]), most, alpha) * o;
             dst[c] = from_f32<T>(v);
         }
     }
@@ -1569,7 +1646,7 @@ expert_combine_kernel(T* __restrict__ act, long ld_act, const T* __restrict__ gu
 
 extern "C" int mllm_hybrid_expert_combine(void* act, long ld_act, const void* gu, long ld_gu, const int* choice,
                                           const float* in_weight, const float* out_weight, int n_experts, int inner, int total,
-                                          int top, int pairs, int gated, float* hidden, long ld_hidden, const void* x, long ld_x,
+                                          int top, int pairs, int form, float limit, float shared_limit, float alpha, float* hidden, long ld_hidden, const void* x, long ld_x,
                                           const float* identity_weight, int width, int assign, int n_tokens, int dtype,
                                           void* stream) {
     if (n_tokens <= 0) return 0;
@@ -1583,36 +1660,46 @@ extern "C" int mllm_hybrid_expert_combine(void* act, long ld_act, const void* gu
     dim3 grid(n_tokens, y);
     const size_t shared = sizeof(float) * 2 * ((size_t)n_experts + 1);
     if (shared > 48 * 1024) return fail("expert_combine: too many experts for the table of weights");
-#define RUN(T, VEC, GATED)                                                                                                      \
-    launch_kernel(g_dependent_launch != 0, expert_combine_kernel<T, VEC, GATED>, grid, dim3(256), shared, s, (T*)act, ld_act,   \
+    if (form < EXPERT_GATED_SILU || form > EXPERT_CLAMPED_GLU) return fail("expert_combine: unknown form of an expert");
+#define RUN(T, VEC, FORM)                                                                                                       \
+    launch_kernel(g_dependent_launch != 0, expert_combine_kernel<T, VEC, FORM>, grid, dim3(256), shared, s, (T*)act, ld_act,    \
                   (const T*)gu, ld_gu, choice, in_weight, out_weight, n_experts, inner, total, top, pairs, hidden, ld_hidden,    \
-                  (const T*)x, ld_x, identity_weight, width, assign)
+                  (const T*)x, ld_x, identity_weight, width, assign, limit, shared_limit, alpha)
+#define PICK(T, VEC)                                                                                                            \
+    do {                                                                                                                        \
+        if (form == EXPERT_GATED_SILU) RUN(T, VEC, EXPERT_GATED_SILU);                                                          \
+        else if (form == EXPERT_RELU_SQUARED) RUN(T, VEC, EXPERT_RELU_SQUARED);                                                 \
+        else RUN(T, VEC, EXPERT_CLAMPED_GLU);                                                                                   \
+    } while (0)
 #define RUN_AS(T)                                                                                                               \
     do {                                                                                                                        \
-        if (vec) { if (gated) RUN(T, true, true); else RUN(T, true, false); }                                                   \
-        else { if (gated) RUN(T, false, true); else RUN(T, false, false); }                                                     \
+        if (vec) PICK(T, true);                                                                                                 \
+        else PICK(T, false);                                                                                                    \
     } while (0)
     if (dtype == DT_F32) RUN_AS(float);
     else RUN_AS(bf16);
 #undef RUN_AS
+#undef PICK
 #undef RUN
     return check_launch("expert_combine_kernel");
 }
 
 extern "C" int mllm_hybrid_route(const void* x, long ld_x, const void* router, const float* router_bias, const float* correction,
                                  const void* shared_gate, int shared_plain, int rule, float scale, int width, int n_outputs,
-                                 int n_identity, int top, int* choice, float* in_weight, float* out_weight,
-                                 float* identity_weight, int n_tokens, int dtype, void* stream) {
+                                 int n_identity, int groups, int keep_groups, int top, int* choice, float* in_weight,
+                                 float* out_weight, float* identity_weight, int n_tokens, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     if (top <= 0 || top > n_outputs) return fail("route: every token takes between one and all experts");
     if (shared_plain && shared_gate != nullptr) return fail("route: the shared expert has a gate or none");
-    if (rule < ROUTE_SIGMOID_ON_INPUT || rule > ROUTE_SOFTMAX_OF_ALL) return fail("route: unknown rule");
+    if (rule < ROUTE_SIGMOID_ON_INPUT || rule > ROUTE_SIGMOID) return fail("route: unknown rule");
+    if (groups < 0 || (groups > 0 && (n_outputs % groups != 0 || keep_groups < 1 || keep_groups > groups || keep_groups * (n_outputs / groups) < top)))
+        return fail("route: equal groups of experts, and enough of them kept to choose from");
     if (n_identity < 0 || n_identity > n_outputs) return fail("route: more identity experts than experts");
     if (n_identity > 0 && (identity_weight == nullptr || rule == ROUTE_SIGMOID_ON_INPUT))
         return fail("route: identity experts need weights on the outputs and room for the token's sum of them");
     cudaStream_t s = (cudaStream_t)stream;
     const int pairs = top + (shared_gate != nullptr || shared_plain ? 1 : 0);
-    const size_t one = sizeof(float) * ((size_t)width + 2 * (size_t)n_outputs + 1);
+    const size_t one = sizeof(float) * ((size_t)width + 2 * (size_t)n_outputs + 1 + (size_t)groups);
     if (one > 48 * 1024) return fail("route: the token and the scores do not fit shared memory");
     const bool four = n_tokens >= 512 && 4 * one <= 48 * 1024;
     // a warp for every output in steps of few tokens, four to sixteen of them
@@ -1620,8 +1707,8 @@ extern "C" int mllm_hybrid_route(const void* x, long ld_x, const void* router, c
 #define RUN(T, TOKENS)                                                                                                          \
     launch_kernel(g_dependent_launch != 0, route_kernel<T, TOKENS>, dim3((n_tokens + TOKENS - 1) / TOKENS), dim3(32 * warps),   \
                   TOKENS * one, s, (const T*)x, ld_x, (const T*)router, router_bias, correction, (const T*)shared_gate,         \
-                  shared_plain, rule, scale, width, n_outputs, n_identity, top, pairs, n_tokens, choice, in_weight, out_weight, \
-                  identity_weight)
+                  shared_plain, rule, scale, width, n_outputs, n_identity, groups, keep_groups, top, pairs, n_tokens, choice,  \
+                  in_weight, out_weight, identity_weight)
     if (dtype == DT_F32) { if (four) RUN(float, 4); else RUN(float, 1); }
     else if (dtype == DT_BF16) { if (four) RUN(bf16, 4); else RUN(bf16, 1); }
     else return fail("route: unknown dtype");
@@ -1629,27 +1716,31 @@ extern "C" int mllm_hybrid_route(const void* x, long ld_x, const void* router, c
     return check_launch("route_kernel");
 }
 
-// (gate_of null: experts without a gate matrix, act = the square of relu; identity_weight: see expert_down)
+// (form: an ExpertForm, with its constants; EXPERT_RELU_SQUARED has no gate matrices; expert `n_experts` is the shared one;
+// identity_weight: see expert_down)
 extern "C" int mllm_hybrid_experts(float* hidden, long ld_hidden, void* act, long ld_act, const void* x, long ld_x,
                                    const int* choice, const float* in_weight, const float* out_weight,
                                    const long long* gate_of, const long long* up_of, const long long* down_of,
                                    const int* inner_of, long ld_down, int max_inner, int width, int pairs,
-                                   const float* identity_weight, int n_tokens, int assign, int dtype, void* stream) {
+                                   const float* identity_weight, int form, float limit, float shared_limit, float alpha,
+                                   int n_experts, int n_tokens, int assign, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
+    if (form < EXPERT_GATED_SILU || form > EXPERT_CLAMPED_GLU || (form != EXPERT_RELU_SQUARED && gate_of == nullptr))
+        return fail("experts: unknown form of an expert, or one without its gate matrices");
     cudaStream_t s = (cudaStream_t)stream;
     const size_t shared = sizeof(float) * (size_t)width;
     if (shared > 48 * 1024) return fail("experts: the token does not fit shared memory");
     constexpr int F = 4, C = 2;
     dim3 up_grid(n_tokens * pairs, (max_inner + 8 * F - 1) / (8 * F)), down_grid(n_tokens, (width + 8 * C - 1) / (8 * C));
     if (up_grid.y > 65535 || down_grid.y > 65535) return fail("experts: the sizes are too large for one launch");
+#define UP(T, FORM)                                                                                                             \
+    launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, FORM, F>, up_grid, dim3(256), shared, s, (T*)act, ld_act,        \
+                  (const T*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs, limit, shared_limit, alpha, n_experts)
 #define RUN(T)                                                                                                                  \
     do {                                                                                                                        \
-        if (gate_of != nullptr)                                                                                                 \
-            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, true, F>, up_grid, dim3(256), shared, s, (T*)act, ld_act, \
-                          (const T*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);                        \
-        else                                                                                                                    \
-            launch_kernel(g_dependent_launch != 0, expert_up_kernel<T, false, F>, up_grid, dim3(256), shared, s, (T*)act, ld_act, \
-                          (const T*)x, ld_x, choice, in_weight, gate_of, up_of, inner_of, width, pairs);                        \
+        if (form == EXPERT_GATED_SILU) UP(T, EXPERT_GATED_SILU);                                                                \
+        else if (form == EXPERT_RELU_SQUARED) UP(T, EXPERT_RELU_SQUARED);                                                       \
+        else UP(T, EXPERT_CLAMPED_GLU);                                                                                         \
         launch_kernel(g_dependent_launch != 0, expert_down_kernel<T, C>, down_grid, dim3(256), 0, s, hidden, ld_hidden,         \
                       (const T*)act, ld_act, choice, out_weight, down_of, inner_of, ld_down, width, pairs, assign, (const T*)x, \
                       ld_x, identity_weight);                                                                                   \
@@ -1658,6 +1749,7 @@ extern "C" int mllm_hybrid_experts(float* hidden, long ld_hidden, void* act, lon
     else if (dtype == DT_BF16) RUN(bf16);
     else return fail("experts: unknown dtype");
 #undef RUN
+#undef UP
     return check_launch("expert kernels");
 }
 

@@ -282,15 +282,16 @@ extern "C" int mllm_sequence_causal_taps(void* out, long ld_out, const void* h, 
 //   product with the key expansion).
 // Rotary positions: among the first rot_dims entries, pair i turns by position * inv_freq[i] and
 // the rest pass unchanged; the pair is (x[2i], x[2i+1]) (layout 0, interleaved) or
-// (x[i], x[i + rot_dims/2]) (layout 1, halves).  Angles in 64-bit.
+// (x[i], x[i + rot_dims/2]) (layout 1, halves).  Angles in 64-bit; cosine and sine are multiplied by
+// `amplitude`.  Rows of `down` lie ld_down apart (other products may stand behind the row).
 // With `writes` false nothing is stored and `down` is not read (it may be null): an entry that
 // reads another entry's rows prepares its queries only.
 // One block per token.
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void latent_prepare_kernel(T* __restrict__ pages, float* __restrict__ q_eff, const float* __restrict__ down,
-                                      const T* __restrict__ q, long ld_q, const float* __restrict__ gain,
-                                      const double* __restrict__ inv_freq, const int* __restrict__ positions,
+                                      long ld_down, const T* __restrict__ q, long ld_q, const float* __restrict__ gain,
+                                      const double* __restrict__ inv_freq, double amplitude, const int* __restrict__ positions,
                                       const int* __restrict__ token_item, const int* __restrict__ block_table,
                                       int max_blocks, int page_size, int rank, int rot, int rot_dims, int heads, int dim,
                                       float eps, int writes, int layout) {
@@ -304,8 +305,8 @@ __global__ void latent_prepare_kernel(T* __restrict__ pages, float* __restrict__
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         double s, c;
         sincos((double)p * inv_freq[i], &s, &c);
-        turn[i] = (float)c;
-        turn[half + i] = (float)s;
+        turn[i] = (float)(c * amplitude);
+        turn[half + i] = (float)(s * amplitude);
     }
     // entry e of a rotated part: its pair's index, its partner, and whether it is the pair's second
     auto pair_of = [&](int e, int& i, int& partner) -> bool {
@@ -317,7 +318,7 @@ __global__ void latent_prepare_kernel(T* __restrict__ pages, float* __restrict__
         return e >= half;
     };
     if (writes) {
-        const float* mine = down + (long)t * (rank + rot);
+        const float* mine = down + (long)t * ld_down;
         float sq = 0.0f;
         for (int d = threadIdx.x; d < rank; d += blockDim.x) sq = fmaf(mine[d], mine[d], sq);
         const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)rank + eps);      // (its barriers also publish turn[])
@@ -351,8 +352,8 @@ __global__ void latent_prepare_kernel(T* __restrict__ pages, float* __restrict__
     }
 }
 
-extern "C" int mllm_sequence_latent_prepare(void* pages, float* q_eff, const float* down, const void* q, long ld_q,
-                                            const float* gain, const double* inv_freq, const int* positions,
+extern "C" int mllm_sequence_latent_prepare(void* pages, float* q_eff, const float* down, long ld_down, const void* q,
+                                            long ld_q, const float* gain, const double* inv_freq, double amplitude, const int* positions,
                                             const int* token_item, const int* block_table, int max_blocks, int page_size,
                                             int n_tokens, int rank, int rot, int rot_dims, int heads, int dim, float eps,
                                             int writes, int layout, int dtype, void* stream) {
@@ -363,11 +364,11 @@ extern "C" int mllm_sequence_latent_prepare(void* pages, float* q_eff, const flo
     cudaStream_t s = (cudaStream_t)stream;
     const size_t shared = (size_t)(rot_dims > 0 ? rot_dims : 1) * sizeof(float);
     if (dtype == DT_F32)
-        launch_kernel(g_dependent_launch != 0, latent_prepare_kernel<float>, dim3(n_tokens), dim3(128), shared, s, (float*)pages, q_eff, down, (const float*)q, ld_q, gain, inv_freq,
+        launch_kernel(g_dependent_launch != 0, latent_prepare_kernel<float>, dim3(n_tokens), dim3(128), shared, s, (float*)pages, q_eff, down, ld_down, (const float*)q, ld_q, gain, inv_freq, amplitude,
                                                                    positions, token_item, block_table, max_blocks, page_size,
                                                                    rank, rot, rot_dims, heads, dim, eps, writes, layout);
     else if (dtype == DT_BF16)
-        launch_kernel(g_dependent_launch != 0, latent_prepare_kernel<bf16>, dim3(n_tokens), dim3(128), shared, s, (bf16*)pages, q_eff, down, (const bf16*)q, ld_q, gain, inv_freq,
+        launch_kernel(g_dependent_launch != 0, latent_prepare_kernel<bf16>, dim3(n_tokens), dim3(128), shared, s, (bf16*)pages, q_eff, down, ld_down, (const bf16*)q, ld_q, gain, inv_freq, amplitude,
                                                                   positions, token_item, block_table, max_blocks, page_size,
                                                                   rank, rot, rot_dims, heads, dim, eps, writes, layout);
     else
@@ -501,14 +502,16 @@ extern "C" int mllm_sequence_head_linear(void* out, const void* a, const void* w
 // value.  The query at position p sees positions 0 .. p of its own request, or the last `window`
 // of them (window <= 0: all).  Four warps take
 // the keys in turn, each with an online softmax (32-bit); their states are merged in a fixed
-// order.  out[t, head, :rank] in 32-bit.  R: 32-element pieces of a row a lane may hold.
+// order.  out[t, head, :rank] in 32-bit, with `gate` times sigmoid(gate[t, head]).  R: 32-element pieces of a row a lane may hold.
 // ---------------------------------------------------------------------------
+__device__ __forceinline__ float gate_open(float z) { return 1.0f / (1.0f + expf(-z)); }
+
 template <typename T, int R>
 __global__ void __launch_bounds__(128)
 latent_attention_kernel(float* __restrict__ out, const float* __restrict__ q_eff, const T* __restrict__ pages,
                         const int* __restrict__ block_table, int max_blocks, const int* __restrict__ positions,
                         const int* __restrict__ token_item, int heads, int rank, int rot, int page_size, float scale,
-                        int window) {
+                        int window, const float* __restrict__ gate, long ld_gate) {
     dependents_may_start();
     wait_for_earlier_kernels();
     const int t = blockIdx.x, h = blockIdx.y;
@@ -560,29 +563,30 @@ latent_attention_kernel(float* __restrict__ out, const float* __restrict__ q_eff
         wgt[w] = sm_m[w] == -INFINITY ? 0.0f : expf(sm_m[w] - big);
         total += sm_l[w] * wgt[w];
     }
+    const float open = gate != nullptr ? gate_open(gate[(long)t * ld_gate + h]) : 1.0f;
     for (int d = threadIdx.x; d < rank; d += blockDim.x) {
         float o = 0.0f;
 #pragma unroll
         for (int w = 0; w < 4; w++) o += sm_acc[w][d] * wgt[w];
-        out[((long)t * heads + h) * rank + d] = o / total;
+        out[((long)t * heads + h) * rank + d] = o / total * open;
     }
 }
 
 template <typename T>
 static int launch_latent_attention(float* out, const float* q_eff, const void* pages, const int* block_table, int max_blocks,
                                    const int* positions, const int* token_item, int n_tokens, int heads, int rank, int rot,
-                                   int page_size, float scale, int window, cudaStream_t s) {
+                                   int page_size, float scale, int window, const float* gate, long ld_gate, cudaStream_t s) {
     dim3 grid(n_tokens, heads);
     const T* pg = (const T*)pages;
     const int pieces = (rank + rot + 31) / 32;
     if (pieces <= 4)
-        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 4>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window);
+        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 4>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window, gate, ld_gate);
     else if (pieces <= 8)
-        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 8>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window);
+        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 8>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window, gate, ld_gate);
     else if (pieces <= 20)
-        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 20>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window);
+        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 20>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window, gate, ld_gate);
     else if (pieces <= 36)
-        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 36>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window);
+        launch_kernel(g_dependent_launch != 0, latent_attention_kernel<T, 36>, dim3(grid), dim3(128), 0, s, out, q_eff, pg, block_table, max_blocks, positions, token_item, heads, rank, rot, page_size, scale, window, gate, ld_gate);
     else
         return fail("latent_attention: a cached row may hold at most 1152 entries");
     return check_launch("latent_attention_kernel");
@@ -591,16 +595,16 @@ static int launch_latent_attention(float* out, const float* q_eff, const void* p
 extern "C" int mllm_sequence_latent_attention(float* out, const float* q_eff, const void* pages, const int* block_table,
                                               int max_blocks, const int* positions, const int* token_item, int n_tokens,
                                               int heads, int rank, int rot, int page_size, float scale, int window,
-                                              int dtype, void* stream) {
+                                              const float* gate, long ld_gate, int dtype, void* stream) {
     if (n_tokens <= 0) return 0;
     if (heads <= 0 || heads > 65535 || rank <= 0 || rot < 0) return fail("latent_attention: bad sizes");
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == DT_F32)
         return launch_latent_attention<float>(out, q_eff, pages, block_table, max_blocks, positions, token_item, n_tokens, heads,
-                                              rank, rot, page_size, scale, window, s);
+                                              rank, rot, page_size, scale, window, gate, ld_gate, s);
     if (dtype == DT_BF16)
         return launch_latent_attention<bf16>(out, q_eff, pages, block_table, max_blocks, positions, token_item, n_tokens, heads,
-                                             rank, rot, page_size, scale, window, s);
+                                             rank, rot, page_size, scale, window, gate, ld_gate, s);
     return fail("latent_attention: unknown dtype");
 }
 
@@ -630,6 +634,8 @@ struct LatentTiledParams {
     int out_bf16;                  // `out` holds bfloat16 (the expansion that follows then runs on the tensor cores)
     int key_buffers;               // 2: the next block of cached rows is copied (cp.async) while this one is used; 1: no room for that
     int window;                    // a query sees the last `window` positions only (<= 0: all)
+    const float* gate;             // [T, >= heads] (rows ld_gate apart) or null: head h's result times sigmoid(gate[t, h])
+    long ld_gate;
 };
 
 template <typename T> struct Chunk4;
@@ -885,7 +891,7 @@ latent_attention_tiled_kernel(LatentTiledParams p) {
 #pragma unroll
                 for (int x = 0; x < 8; x++) o[x] = empty ? 0.0f : acc[i][ct * 8 + x];
             } else {
-                const float inv = 1.0f / sums[r];
+                const float inv = (p.gate != nullptr ? gate_open(p.gate[(long)(first_row + token) * p.ld_gate + head]) : 1.0f) / sums[r];
                 if (p.out_bf16) {
                     bf16* o = reinterpret_cast<bf16*>(p.out) + at * p.rank + c0;
 #pragma unroll
@@ -906,7 +912,8 @@ latent_attention_tiled_kernel(LatentTiledParams p) {
 
 // The parts of a (token, head) into one result, in the order of the parts.
 __global__ void latent_merge_kernel(void* __restrict__ out, int out_bf16, const float* __restrict__ part_out,
-                                    const float* __restrict__ part_ml, int parts, int rank) {
+                                    const float* __restrict__ part_ml, int parts, int rank, int heads,
+                                    const float* __restrict__ gate, long ld_gate) {
     dependents_may_start();
     wait_for_earlier_kernels();
     __shared__ float weight[32];                 // of each part (there are at most 32), already divided by the sum
@@ -918,7 +925,8 @@ __global__ void latent_merge_kernel(void* __restrict__ out, int out_bf16, const 
         const float big = warp_max(m);
         const float w = m == -INFINITY ? 0.0f : expf(m - big);
         const float total = warp_sum(l * w);
-        weight[z] = w / total;
+        const float open = gate != nullptr ? gate_open(gate[at / heads * ld_gate + at % heads]) : 1.0f;
+        weight[z] = w / total * open;
     }
     __syncthreads();
     const float* mine = part_out + at * parts * rank;
@@ -990,7 +998,8 @@ extern "C" int mllm_sequence_latent_attention_tiled(const LatentTiledParams* par
     else if (dtype == DT_BF16) rc = pick_latent_tiled<bf16>(p, rows, keys, grid, shared, s);
     else return fail("latent_attention_tiled: unknown dtype");
     if (rc != 0 || p.parts == 1) return rc;
-    launch_kernel(g_dependent_launch != 0, latent_merge_kernel, dim3((unsigned)((long)n_units * p.heads)), dim3(128), 0, s, p.out, p.out_bf16, p.part_out, p.part_ml, p.parts, p.rank);
+    launch_kernel(g_dependent_launch != 0, latent_merge_kernel, dim3((unsigned)((long)n_units * p.heads)), dim3(128), 0, s, p.out, p.out_bf16, p.part_out, p.part_ml, p.parts, p.rank, p.heads,
+                  p.gate, p.ld_gate);
     return check_launch("latent_merge_kernel");
 }
 

@@ -194,6 +194,8 @@ class StepContext:
         self.item_slot = self.item_offset = self.item_count = self.item_start = None    # the same, on the device (int32)
         self.kept_results = None      # fp32 [T, planes, width]: the embedding output and every layer's result, if the model keeps them
         self.streams = None           # fp32 [T, streams, width]: the residual of a model with several residual streams
+        self.next_norm = None         # the norm that reads the stream first in the next run entry, where it is known
+        self.normed_ahead = None      # (that norm, its rows) once a pass over the stream has applied it
         self.streams_pending = None   # a layer's last write onto the streams, waiting to go with the next read-out
         self.decode_only = False      # every entry brings exactly one token
         self.fused = False            # the step goes to the one-kernel decode step

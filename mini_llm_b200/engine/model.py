@@ -2,7 +2,8 @@
 
 Nothing here names an architecture.  ``Model`` builds every part the
 description lists, loads the tensors they declare, and runs a step: embed,
-the run entries in their order (each with the cache view of its entry), then
+the run entries in their order (each with the cache view of its entry; an embedding that keeps
+something per request has the view behind theirs), then
 the final norm and the head on the rows whose logits are wanted only (the
 reference norms and multiplies the last row only,
 engine/src/gpt2_gpu.cu:254-263).
@@ -80,6 +81,9 @@ class Model:
                 needs.append(mine[arrangement.mixer_role()])
             else:
                 needs.append(mine)
+        # an embedding that keeps something owns the entry behind the run entries
+        if not isinstance(self.embedding.cache_need(), NoCache):
+            needs.append(self.embedding.cache_need())
         return needs
 
     def load(self, model_dir: str, dtype, device, runtime=None):
@@ -91,9 +95,17 @@ class Model:
                                 {t.data_ptr(): t for t in tensors.values()}.values())
         return self
 
+    def _first_norm(self, index):
+        """The norm that reads the stream first in run entry ``index``, if its arrangement says so."""
+        if index >= len(self.spec.order):
+            return None
+        arrangement, parts = self.layers[self.spec.order[index].layer]
+        return parts.get(arrangement.first_norm) if arrangement.first_norm is not None else None
+
     def forward(self, ctx, cache_views):
         """Run the step's tokens; returns fp32 logits [n_want, vocab] or None."""
-        hidden = self.embedding.forward(ctx, self.position)
+        kept = {"cache": cache_views[len(self.spec.order)]} if len(cache_views) > len(self.spec.order) else {}
+        hidden = self.embedding.forward(ctx, self.position, **kept)
         if self.embedding_norm is not None:
             self.embedding_norm.normalize_in_place(ctx, hidden)
         ctx.kept_results = None
@@ -111,8 +123,10 @@ class Model:
         dump = getattr(ctx, "dump", None)
         if dump is not None:
             dump.append(hidden.clone())
+        ctx.normed_ahead = None          # (norm part, its rows) where the pass that changed the stream last applied the next norm
         for index, entry in enumerate(self.spec.order):
             arrangement, parts = self.layers[entry.layer]
+            ctx.next_norm = self._first_norm(index + 1)
             arrangement.run(ctx, parts, hidden, cache_views[index])
             if dump is not None:
                 if ctx.streams is not None:

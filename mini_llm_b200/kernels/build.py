@@ -45,6 +45,7 @@ LIBRARIES = {
     "hybrid": "hybrid_kernels.cu",
     "streams": "stream_kernels.cu",
     "unit": "recurrent_unit_kernels.cu",
+    "token": "token_kernels.cu",
 }
 
 _lock = threading.Lock()

@@ -124,11 +124,12 @@ class Kernels:
                                    cache.block_table, cache.page_size, cache.k_pages, cache.v_pages, cache.writes)
 
     def capped_attention(self, ctx, out, q, cache, n_heads, n_kv_heads, dim, vdim, scale, cap=0.0, window=0, chunk=0,
-                         gate=None, sink=None, keep=0):
+                         gate=None, sink=None, keep=0, slopes=None, gate_wide=False):
         """Attention whose weights stay 32-bit, with a cap on the scores and values of a size of
         their own; the mask is causal, over the last ``window`` positions (and the first ``keep``) or within
-        blocks of ``chunk`` positions; ``gate`` [T, heads] opens each head's result by its sigmoid; ``sink`` [heads] adds
-        exp(sink[h]) to head h's denominator.  Steps with
+        blocks of ``chunk`` positions; ``gate`` [T, heads] opens each head's result by its sigmoid (``gate_wide``:
+        [T, heads * vdim], each entry of it); ``sink`` [heads] adds exp(sink[h]) to head h's denominator; ``slopes`` [heads]
+        take slopes[h] * (query's position - key's position) off the score.  Steps with
         prompt portions take the tiles (tokens of a request side by side share the cached rows they
         read); steps of single tokens, and sizes the tiles do not take, one block per (token, head)."""
         self.launches += 1
@@ -147,11 +148,13 @@ class Kernels:
             self.chose("capped_attention", "split_attention", n, n_heads, dim, vdim)
             return ops.split_attention(out, q, cache.k_pages, cache.v_pages, cache.block_table, ctx.positions, ctx.token_item,
                                        n_heads, n_kv_heads, dim, cache.page_size, scale, window, span, -(-reach // span), acc,
-                                       ml, counters, cap=cap, block=chunk, gate=gate, sink=sink, value_size=vdim, keep=keep)
+                                       ml, counters, cap=cap, block=chunk, gate=gate, sink=sink, value_size=vdim, keep=keep, slopes=slopes,
+                                       gate_wide=gate_wide)
         tiled = not ctx.decode_only and ops.capped_attention_tiled_takes(dim, vdim, q.dtype)
         self.chose("capped_attention", "capped_attention_tiled" if tiled else "capped_attention_plain", q.shape[0], n_heads, dim, vdim)
         return ops.capped_attention(out, q, cache.k_pages, cache.v_pages, cache.block_table, ctx.positions, ctx.token_item,
-                                    n_heads, n_kv_heads, dim, vdim, cache.page_size, scale, cap, window, tiled, chunk, gate, sink, keep)
+                                    n_heads, n_kv_heads, dim, vdim, cache.page_size, scale, cap, window, tiled, chunk, gate, sink, keep,
+                                    slopes, gate_wide)
 
     def linear_recurrence(self, ctx, out, q, k, v, gate_a, gate_b, log_rate, step_bias, state, heads, qk_heads, dim, vdim,
                           delta, unit_norm=False, q_scale=1.0, skip=None, writes=True, channel_decay=False):
@@ -165,10 +168,10 @@ class Kernels:
         return ops.route(x, router, shared_gate, top, choice, in_weight, out_weight, **how)
 
     def experts(self, hidden, act, x, choice, in_weight, out_weight, gate_of, up_of, down_of, inner_of, max_inner, pairs,
-                ld_down=None, assign=False, identity_weight=None):
+                ld_down=None, assign=False, identity_weight=None, **form):
         self.launches += 2
         return ops.experts(hidden, act, x, choice, in_weight, out_weight, gate_of, up_of, down_of, inner_of, max_inner, pairs,
-                           ld_down, assign, identity_weight)
+                           ld_down, assign, identity_weight, **form)
 
     EXPERTS_AT_ONCE_TOKENS = 32    # from here on a step's tokens go through all experts as two products
 
@@ -217,10 +220,11 @@ class Kernels:
         return ops.scaled_add(x, u, a, v, b, assign)
 
     def latent_prepare(self, ctx, cache, q_eff, down, q, gain, inv_freq, rank, rot, rot_dims, heads, dim, eps,
-                       layout="interleaved"):
+                       layout="interleaved", amplitude=1.0):
         self.launches += 1
         return ops.latent_prepare(cache.k_pages, q_eff, down, q, gain, inv_freq, ctx.positions, ctx.token_item,
-                                  cache.block_table, cache.page_size, rank, rot, rot_dims, heads, dim, eps, cache.writes, layout)
+                                  cache.block_table, cache.page_size, rank, rot, rot_dims, heads, dim, eps, cache.writes, layout,
+                                  amplitude)
 
     HEAD_LINEAR_GEMM_ROWS = 128   # from here on each head's product goes to the tensor-core kernel by itself
 
@@ -246,7 +250,7 @@ class Kernels:
         tiled = not self.plain_only and ops.latent_attention_tiled_takes(cache.k_pages, rank, rot)
         return torch.bfloat16 if tiled and self.act_dtype == torch.bfloat16 else torch.float32
 
-    def latent_attention(self, ctx, out, q_eff, cache, heads, rank, rot, scale, window=0):
+    def latent_attention(self, ctx, out, q_eff, cache, heads, rank, rot, scale, window=0, gate=None):
         self.launches += 1
         n = q_eff.shape[0]
         if not self.plain_only and ops.latent_attention_tiled_takes(cache.k_pages, rank, rot):
@@ -255,7 +259,7 @@ class Kernels:
             if ctx.att_tiles is not None:
                 # prompt portions: 32 rows (tokens x heads) a block share every cached row they read
                 self.chose("latent_attention", "latent_attention_tiled", n, heads, rank + rot)
-                return ops.latent_attention_tiled(*common, tiles=ctx.att_tiles, n_tiles=ctx.n_att_tiles, window=window)
+                return ops.latent_attention_tiled(*common, tiles=ctx.att_tiles, n_tiles=ctx.n_att_tiles, window=window, gate=gate)
             if ctx.decode_only:
                 # single tokens: all heads of a token share the cached rows; while the (token, head
                 # block) pairs are fewer than twice the SMs, each token's keys come in parts
@@ -264,11 +268,11 @@ class Kernels:
                 scratch = self._latent_scratch(ctx.device, n * heads * parts * rank, n * heads * parts * 2) if parts > 1 else None
                 self.launches += 1 if parts > 1 else 0
                 self.chose("latent_attention", "latent_attention_tiled_parts", n, heads, rank + rot)
-                return ops.latent_attention_tiled(*common, parts=parts, scratch=scratch, window=window)
+                return ops.latent_attention_tiled(*common, parts=parts, scratch=scratch, window=window, gate=gate)
         self.chose("latent_attention", "latent_attention_plain", n, heads, rank + rot)
         plain_out = out if out.dtype == torch.float32 else ctx.buffer("latent_mixed_32", out.shape, torch.float32)
         ops.latent_attention_plain(plain_out, q_eff, cache.k_pages, cache.block_table, ctx.positions, ctx.token_item,
-                                   heads, rank, rot, cache.page_size, scale, window)
+                                   heads, rank, rot, cache.page_size, scale, window, gate)
         if plain_out is not out:
             out.copy_(plain_out)
         return out
@@ -313,6 +317,40 @@ class Kernels:
     def depth_mix(self, hidden, kept, weights, index):
         self.launches += 1
         return ops.depth_mix(hidden, kept, weights, index)
+
+    # ---- what a token's identity adds beyond its embedding row ------------------------------------
+    def pair_embed(self, ctx, out, table, pairs, state, buckets, mul_prev, mul_cur, scale=1.0):
+        self.launches += 1
+        return ops.pair_embed(out, ctx.token_ids, ctx.positions, ctx.token_item, ctx.item_slot, ctx.item_offset, ctx.item_count,
+                              table, pairs, state, buckets, mul_prev, mul_cur, scale)
+
+    TOKEN_GATE_TOKENS = 64         # up to here the gate's product, its gelu and the token's row are one kernel on the stream itself
+
+    def token_gate(self, ctx, out, hidden, w, side, first):
+        """out[t, j] = gelu_tanh(w[j] . hidden[t]) * side[id_t, first + j]."""
+        n, width = hidden.shape
+        if n <= self.TOKEN_GATE_TOKENS and width <= ops.ROW_IN_SHARED_MEMORY:
+            self.launches += 1
+            self.chose("token_gate", "token_gate", n, out.shape[1], width)
+            return ops.token_gate(out, hidden, w, side, ctx.token_ids, first)
+        x = hidden
+        if self.act_dtype != hidden.dtype:
+            x = ctx.buffer("stream_rounded", (n, width), self.act_dtype)
+            self.add_normed_cast(hidden, act=x)
+        z = ctx.buffer("token_gate", tuple(out.shape), torch.float32)
+        self.linear(ctx, z, x, w)
+        self.launches += 1
+        self.chose("token_gate", "token_gate_rows", n, out.shape[1], width)
+        return ops.token_gate_rows(out, z, side, ctx.token_ids, first)
+
+    def add_normed_norm(self, ctx, hidden, y, gain, eps, normed, next_gain, next_eps):
+        """The normed ``y`` onto the stream, then the norm of the rows as they are: one pass where a row fits shared memory."""
+        if hidden.shape[1] <= ops.ROW_IN_SHARED_MEMORY:
+            self.launches += 1
+            return ops.add_normed_norm(hidden, y, gain, eps, normed, next_gain, next_eps)
+        self.add_normed_cast(hidden, y, gain, eps)
+        self.grouped_rms_norm(normed, hidden, next_gain, 1, next_eps)
+        return hidden
 
     def kv_store(self, k_pages, v_pages, k_src, v_src, positions, token_item, block_table, page_size):
         self.launches += 1

@@ -229,7 +229,7 @@ class _SkinnyParams(ctypes.Structure):
 
 _skinny = Function("decode", "mllm_decode_skinny_linear", [ctypes.POINTER(_SkinnyParams), P])
 _split_attention = Function("decode", "mllm_decode_split_attention_kept",
-                            [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, F, I, I, I, P, L, P, I, I, P, P, P, P])
+                            [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, F, I, I, I, P, L, I, P, P, I, I, P, P, P, P])
 
 SKINNY_MAX_SMEM = 200 * 1024
 SPLIT_ATTENTION_HEAD_SIZES = (16, 32, 64, 128, 256)
@@ -312,13 +312,15 @@ def skinny_linear(out, x, w, bias=None, epilogue="store", norm=None, scatter=Non
 
 def split_attention(out, q, k_pages, v_pages, block_table, positions, token_item, n_heads, n_kv_heads, head_size,
                     page_size, scale, window, chunk, max_chunks, part_acc, part_ml, counters, cap=0.0, block=0, gate=None, sink=None,
-                    value_size=None, keep=0):
+                    value_size=None, keep=0, slopes=None, gate_wide=False):
     """Causal attention over the paged cache for few tokens: one CTA per (token, head, chunk
     of ``chunk`` keys); needs fp32 scratch ``part_acc`` [T*H*max_chunks*D], ``part_ml``
     [T*H*max_chunks*2] and zeroed int32 ``counters`` [T*H] (left zero).  ``cap`` > 0: the scores
     are capped, cap * tanh(score / cap).  ``block`` > 0: a query sees only the keys of its own block of
     ``block`` positions (blocks counted from position 0).  ``gate`` fp32 [T, >= heads]: head h's result
-    is multiplied by sigmoid(gate[t, h]).  ``sink`` fp32 [heads]: exp(sink[h]) joins head h's denominator.
+    is multiplied by sigmoid(gate[t, h]); with ``gate_wide`` [T, >= heads * value_size] every entry of the result by its own.
+    ``sink`` fp32 [heads]: exp(sink[h]) joins head h's denominator.  ``slopes`` fp32 [heads]: slopes[h] * (query's position -
+    key's position) comes off the (capped) score.
     ``value_size``: entries of a value where they are not ``head_size`` (then both are multiples of 8 up to 256 and the
     scratch is sized for ``split_attention_row``).  ``keep``: the first ``keep`` keys stay visible behind the window.
     ``max_chunks`` chunks must cover the most keys a token may see.  Scores, weights and sums are 32-bit."""
@@ -345,24 +347,29 @@ def split_attention(out, q, k_pages, v_pages, block_table, positions, token_item
         raise KernelError("split_attention: the chunks do not cover the longest block table (or the window)")
     if keep < 0 or (keep and block):
         raise KernelError("split_attention: kept first keys go with a window, not with blocks of positions")
-    if gate is not None:
-        _check(gate, "split_attention.gate", torch.float32, 2)
-        if gate.shape[0] < n or gate.shape[1] < n_heads or gate.stride(1) != 1:
-            raise KernelError("split_attention: one gate per token and head")
-    _check_sink(sink, n_heads, "split_attention")
+    _check_gate(gate, n, n_heads * (vdim if gate_wide else 1), "split_attention")
+    _check_per_head(sink, n_heads, "split_attention.sink")
+    _check_per_head(slopes, n_heads, "split_attention.slopes")
     _split_attention(out.data_ptr(), out.stride(0), q.data_ptr(), q.stride(0), k_pages.data_ptr(), v_pages.data_ptr(),
                      block_table.data_ptr(), block_table.shape[1], positions.data_ptr(), token_item.data_ptr(), n,
                      n_heads, n_kv_heads, head_size, vdim, page_size, float(scale), float(cap or 0.0), int(window or 0), int(block or 0),
-                     int(keep), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(sink), int(chunk), int(max_chunks), part_acc.data_ptr(),
+                     int(keep), _ptr(gate), gate.stride(0) if gate is not None else 0, int(bool(gate_wide)), _ptr(sink), _ptr(slopes), int(chunk), int(max_chunks), part_acc.data_ptr(),
                      part_ml.data_ptr(), counters.data_ptr(), _stream())
     return out
 
 
-def _check_sink(sink, n_heads, who):
-    if sink is not None:
-        _check(sink, f"{who}.sink", torch.float32, 1)
-        if sink.shape[0] != n_heads:
-            raise KernelError(f"{who}: one sink per head")
+def _check_per_head(values, n_heads, who):
+    if values is not None:
+        _check(values, who, torch.float32, 1)
+        if values.shape[0] != n_heads:
+            raise KernelError(f"{who}: one number per head")
+
+
+def _check_gate(gate, n, columns, who):
+    if gate is not None:
+        _check(gate, f"{who}.gate", torch.float32, 2)
+        if gate.shape[0] < n or gate.shape[1] < columns or gate.stride(1) != 1:
+            raise KernelError(f"{who}: the gate has fewer rows than tokens, or not {columns} columns")
 
 
 _group_attention = Function("decode", "mllm_decode_group_attention",
@@ -915,18 +922,19 @@ def norm_taps_step(out, x, gain, groups, eps, w, state, token_item, item_slot, w
 
 
 _latent_prepare = Function("sequence", "mllm_sequence_latent_prepare",
-                           [P, P, P, P, L, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P])
+                           [P, P, P, L, P, L, P, P, ctypes.c_double, P, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P])
 ROTARY_LAYOUTS = {"interleaved": 0, "half": 1}
 
 
 def latent_prepare(pages, q_eff, down, q, gain, inv_freq, positions, token_item, block_table, page_size, rank, rot,
-                   rot_dims, heads, dim, eps, writes=True, layout="interleaved"):
+                   rot_dims, heads, dim, eps, writes=True, layout="interleaved", amplitude=1.0):
     """Per token: the first ``rank`` entries of the fp32 ``down`` row, normed by their root mean square
     and times ``gain``, and its last ``rot`` entries with rotary positions, go into the token's row
     of ``pages`` [n_pages, page_size, 1, rank + rot]; the rotated part of every head's query
     (``q`` [T, heads * (dim + rot)]) gets rotary positions and goes to
     ``q_eff`` [T, heads * (rank + rot)] (fp32), entries rank .. rank + rot of each head.  ``layout``: the
     pairs that turn together are neighbours ("interleaved") or half the rotated entries apart ("half").
+    Cosine and sine are multiplied by ``amplitude``.  ``down`` may be the first columns of a wider buffer.
     With ``writes`` false only the queries are prepared and ``down`` may be None."""
     _check(pages, "latent_prepare.pages", q.dtype)
     _check(q_eff, "latent_prepare.q_eff", torch.float32, 2)
@@ -941,13 +949,13 @@ def latent_prepare(pages, q_eff, down, q, gain, inv_freq, positions, token_item,
     _check(block_table, "latent_prepare.block_table", torch.int32, 2)
     n = q.shape[0]
     row = rank + rot
-    if (not down.is_contiguous() or down.shape[1] != row or not q_eff.is_contiguous() or q_eff.shape[1] != heads * row
+    if (down.shape[1] != row or down.stride(1) != 1 or not q_eff.is_contiguous() or q_eff.shape[1] != heads * row
             or q.shape[1] != heads * (dim + rot) or gain.shape[0] != rank or inv_freq.shape[0] < rot_dims // 2):
         raise KernelError("latent_prepare: sizes do not agree")
     if not pages.is_contiguous() or pages.numel() % (page_size * row) != 0 or not block_table.is_contiguous():
         raise KernelError("latent_prepare: the pages do not hold whole pages of rows of rank + rot")
-    _latent_prepare(pages.data_ptr(), q_eff.data_ptr(), down.data_ptr() if down.numel() else None, q.data_ptr(), q.stride(0), gain.data_ptr(),
-                    inv_freq.data_ptr(), positions.data_ptr(), token_item.data_ptr(), block_table.data_ptr(),
+    _latent_prepare(pages.data_ptr(), q_eff.data_ptr(), down.data_ptr() if down.numel() else None, down.stride(0), q.data_ptr(), q.stride(0),
+                    gain.data_ptr(), inv_freq.data_ptr(), float(amplitude), positions.data_ptr(), token_item.data_ptr(), block_table.data_ptr(),
                     block_table.shape[1], page_size, n, rank, rot, rot_dims, heads, dim, float(eps), int(bool(writes)),
                     ROTARY_LAYOUTS[layout], dtype_code(q.dtype), _stream())
 
@@ -971,14 +979,15 @@ def head_linear(out, a, w, heads, a_head, o_head):
     return out
 
 
-_latent_attention = Function("sequence", "mllm_sequence_latent_attention", [P, P, P, P, I, P, P, I, I, I, I, I, F, I, I, P])
+_latent_attention = Function("sequence", "mllm_sequence_latent_attention", [P, P, P, P, I, P, P, I, I, I, I, I, F, I, P, L, I, P])
+
 
 
 def latent_attention_plain(out, q_eff, pages, block_table, positions, token_item, heads, rank, rot, page_size, scale,
-                           window=0):
+                           window=0, gate=None):
     """Causal attention of every token of the step over its request's cached rows [rank + rot]:
     score = q_eff[t, head] . row * scale, value = the row's first ``rank`` entries;
-    out [T, heads * rank] in 32-bit."""
+    out [T, heads * rank] in 32-bit.  ``gate`` fp32 [T, >= heads]: head h's result is multiplied by sigmoid(gate[t, h])."""
     _check(out, "latent_attention.out", torch.float32, 2)
     _check(q_eff, "latent_attention.q_eff", torch.float32, 2)
     _check(pages, "latent_attention.pages")
@@ -987,9 +996,10 @@ def latent_attention_plain(out, q_eff, pages, block_table, positions, token_item
     if (not out.is_contiguous() or not q_eff.is_contiguous() or out.shape != (n, heads * rank)
             or q_eff.shape[1] != heads * (rank + rot) or not pages.is_contiguous() or not block_table.is_contiguous()):
         raise KernelError("latent_attention: sizes do not agree")
+    _check_gate(gate, n, heads, "latent_attention")
     _latent_attention(out.data_ptr(), q_eff.data_ptr(), pages.data_ptr(), block_table.data_ptr(), block_table.shape[1],
                       positions.data_ptr(), token_item.data_ptr(), n, heads, rank, rot, page_size, float(scale),
-                      int(window or 0), dtype_code(pages.dtype), _stream())
+                      int(window or 0), _ptr(gate), gate.stride(0) if gate is not None else 0, dtype_code(pages.dtype), _stream())
     return out
 
 
@@ -997,7 +1007,7 @@ class _LatentTiledParams(ctypes.Structure):
     _fields_ = [("out", P), ("part_out", P), ("part_ml", P), ("q_eff", P), ("pages", P), ("block_table", P),
                 ("positions", P), ("token_item", P), ("tiles", P), ("max_blocks", I), ("page_size", I), ("n_tokens", I),
                 ("heads", I), ("rank", I), ("rot", I), ("TQ", I), ("HB", I), ("parts", I),
-                ("scale", F), ("out_bf16", I), ("key_buffers", I), ("window", I)]
+                ("scale", F), ("out_bf16", I), ("key_buffers", I), ("window", I), ("gate", P), ("ld_gate", L)]
 
 
 _latent_attention_tiled = Function("sequence", "mllm_sequence_latent_attention_tiled",
@@ -1022,12 +1032,12 @@ def latent_heads_per_block(heads: int) -> int:
 
 
 def latent_attention_tiled(out, q_eff, pages, block_table, positions, token_item, heads, rank, rot, page_size, scale,
-                           tiles=None, n_tiles=0, parts=1, scratch=None, window=0):
+                           tiles=None, n_tiles=0, parts=1, scratch=None, window=0, gate=None):
     """``latent_attention_plain`` in tiles of 32 query rows that share their keys.  With ``tiles``
     (the step's work list, device int32 records of 8, ``n_tiles`` of them) for prompt portions;
     without, for single tokens, the keys of each in ``parts`` runs (the token's context length over
     ``parts``, in whole blocks of 32) whose results are merged (``scratch``: fp32 (T * heads * parts * rank, T * heads * parts * 2)).
-    ``out`` may be bfloat16: the sums are 32-bit either way, the result is rounded once."""
+    ``out`` may be bfloat16: the sums are 32-bit either way, the result is rounded once.  ``gate`` as in the plain form."""
     _check(out, "latent_attention.out", None, 2)
     if out.dtype not in (torch.float32, torch.bfloat16):
         raise KernelError("latent_attention_tiled: out must be float32 or bfloat16")
@@ -1047,6 +1057,8 @@ def latent_attention_tiled(out, q_eff, pages, block_table, positions, token_item
     params.heads, params.rank, params.rot, params.scale = heads, rank, rot, float(scale)
     params.out_bf16 = int(out.dtype == torch.bfloat16)
     params.window = int(window or 0)           # (> 0: a query sees the last ``window`` positions only)
+    _check_gate(gate, n, heads, "latent_attention")
+    params.gate, params.ld_gate = _ptr(gate), gate.stride(0) if gate is not None else 0
     if tiles is not None:
         _check(tiles, "latent_attention.tiles", torch.int32)
         if tiles.numel() < ATTENTION_TILE_RECORD * n_tiles or parts != 1:
@@ -1217,7 +1229,7 @@ def rotary_store(qkv, k_off, v_off, heads, kv_heads, dim, vdim, rot_dims, inv_fr
 
 
 _capped_attention = Function("hybrid", "mllm_hybrid_capped_attention",
-                             [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, F, I, I, I, P, L, P, I, I, P])
+                             [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, F, I, I, I, P, L, I, P, P, I, I, P])
 
 
 def capped_attention_tiled_takes(dim, vdim, dtype=torch.bfloat16) -> bool:
@@ -1230,13 +1242,16 @@ def capped_attention_tiled_takes(dim, vdim, dtype=torch.bfloat16) -> bool:
 
 
 def capped_attention(out, q, k_pages, v_pages, block_table, positions, token_item, n_heads, n_kv_heads, dim, vdim,
-                     page_size, scale, cap=0.0, window=0, tiled=False, chunk=0, gate=None, sink=None, keep=0):
+                     page_size, scale, cap=0.0, window=0, tiled=False, chunk=0, gate=None, sink=None, keep=0, slopes=None,
+                     gate_wide=False):
     """Causal attention of every token of the step over its request's pages, keys of ``dim`` and
     values of ``vdim`` entries per head, score = cap * tanh(q . k * scale / cap) (``cap`` 0: no cap);
     scores, weights and the weighted sum in 32-bit.  ``window`` > 0: the last ``window`` positions only, and the
     first ``keep`` of the sequence; ``chunk`` > 0: only keys of the query's own block of ``chunk`` positions (blocks counted from
-    position 0).  ``gate`` fp32 [T, >= heads]: head h's result is multiplied by sigmoid(gate[t, h]).
+    position 0).  ``gate`` fp32 [T, >= heads]: head h's result is multiplied by sigmoid(gate[t, h]); with ``gate_wide``
+    [T, >= heads * vdim] every entry of the result by its own.
     ``sink`` fp32 [heads]: the softmax's denominator also holds exp(sink[h]), a term with no key and no value.
+    ``slopes`` fp32 [heads]: slopes[h] * (query's position - key's position) comes off the (capped) score.
     ``tiled``: consecutive tokens of a request share the cached rows they read (for steps with prompt
     portions)."""
     _check(out, "capped_attention.out", q.dtype, 2)
@@ -1249,18 +1264,16 @@ def capped_attention(out, q, k_pages, v_pages, block_table, positions, token_ite
         raise KernelError("capped_attention: q / out do not have heads * size columns")
     if not k_pages.is_contiguous() or not v_pages.is_contiguous() or not block_table.is_contiguous():
         raise KernelError("capped_attention: pages and block table must be contiguous")
-    if gate is not None:
-        _check(gate, "capped_attention.gate", torch.float32, 2)
-        if gate.shape[0] < n or gate.shape[1] < n_heads or gate.stride(1) != 1:
-            raise KernelError("capped_attention: one gate per token and head")
-    _check_sink(sink, n_heads, "capped_attention")
+    _check_gate(gate, n, n_heads * (vdim if gate_wide else 1), "capped_attention")
+    _check_per_head(sink, n_heads, "capped_attention.sink")
+    _check_per_head(slopes, n_heads, "capped_attention.slopes")
     if keep < 0 or (keep and chunk):
         raise KernelError("capped_attention: kept first keys go with a window, not with blocks of positions")
     _capped_attention(out.data_ptr(), out.stride(0), q.data_ptr(), q.stride(0), k_pages.data_ptr(), v_pages.data_ptr(),
                       block_table.data_ptr(), block_table.shape[1], positions.data_ptr(), token_item.data_ptr(), n, n_heads,
                       n_kv_heads, dim, vdim, page_size, float(scale), float(cap or 0.0), int(window or 0), int(chunk or 0),
-                      int(keep), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(sink), int(bool(tiled)), dtype_code(q.dtype),
-                      _stream())
+                      int(keep), _ptr(gate), gate.stride(0) if gate is not None else 0, int(bool(gate_wide)), _ptr(sink), _ptr(slopes), int(bool(tiled)),
+                      dtype_code(q.dtype), _stream())
     return out
 
 
@@ -1344,22 +1357,26 @@ def linear_recurrence(out, q, k, v, gate_a, gate_b, log_rate, step_bias, state, 
     return out
 
 
-_route = Function("hybrid", "mllm_hybrid_route", [P, L, P, P, P, P, I, I, F, I, I, I, I, P, P, P, P, I, I, P])
-_experts = Function("hybrid", "mllm_hybrid_experts", [P, L, P, L, P, L, P, P, P, P, P, P, P, L, I, I, I, P, I, I, I, P])
+_route = Function("hybrid", "mllm_hybrid_route", [P, L, P, P, P, P, I, I, F, I, I, I, I, I, I, P, P, P, P, I, I, P])
+_experts = Function("hybrid", "mllm_hybrid_experts", [P, L, P, L, P, L, P, P, P, P, P, P, P, L, I, I, I, P, I, F, F, F, I, I, I, I, P])
 _expert_combine = Function("hybrid", "mllm_hybrid_expert_combine",
-                           [P, L, P, L, P, P, P, I, I, I, I, I, I, P, L, P, L, P, I, I, I, I, P])
-ROUTE_RULES = {"sigmoid_on_input": 0, "softmax_of_chosen": 1, "softmax_of_all": 2}
+                           [P, L, P, L, P, P, P, I, I, I, I, I, I, F, F, F, P, L, P, L, P, I, I, I, I, P])
+ROUTE_RULES = {"sigmoid_on_input": 0, "softmax_of_chosen": 1, "softmax_of_all": 2, "sigmoid": 3}
+EXPERT_FORMS = {"gated_silu": 0, "relu_squared": 1, "clamped_glu": 2}
 
 
 def route(x, router, shared_gate, top, choice, in_weight, out_weight, bias=None, rule="sigmoid_on_input", shared_plain=False,
-          correction=None, n_identity=0, scale=1.0, identity_weight=None):
+          correction=None, n_identity=0, scale=1.0, identity_weight=None, groups=0, keep_groups=0):
     """Per row of ``x``: the outputs of ``router`` [outputs, width] (sums in 32-bit, plus ``bias`` fp32 [outputs]), of which the
     ``top`` largest are chosen (the lower index wins a tie).  ``rule``:
     "sigmoid_on_input": sigmoid scores rank them and weigh the chosen experts' inputs;
     "softmax_of_chosen": the logits rank them; the chosen ones get input weight 1 and, as output weight, the softmax over
     the chosen logits only;
     "softmax_of_all": s = the softmax over all outputs; s + ``correction`` (fp32 [outputs]) ranks them; output weights
-    s / (sum of the chosen s + 1e-20) * ``scale``.
+    s / (sum of the chosen s + 1e-20) * ``scale``;
+    "sigmoid": s = the sigmoids; s + ``correction`` ranks them; output weights s * ``scale``.
+    With ``groups`` the outputs form that many equal runs of neighbours and only those of the ``keep_groups`` best can be
+    chosen; a group's score is the sum of its two largest ranking scores.
     The last ``n_identity`` outputs are identity experts (the output is the token itself): such a choice is stored as
     -1 with weight 0, and the token's weights of that kind are summed in ``identity_weight`` fp32 [T].
     With ``shared_gate`` [1, width] one more pair per token: expert ``outputs - n_identity``, input weight 1, output weight
@@ -1390,7 +1407,7 @@ def route(x, router, shared_gate, top, choice, in_weight, out_weight, bias=None,
         if shared_gate.numel() != width or not shared_gate.is_contiguous():
             raise KernelError("route: the shared expert's gate is one row of the width")
     _route(x.data_ptr(), x.stride(0), router.data_ptr(), _ptr(bias), _ptr(correction), _ptr(shared_gate), int(bool(shared_plain)),
-           ROUTE_RULES[rule], float(scale), width, router.shape[0], int(n_identity), top, choice.data_ptr(), in_weight.data_ptr(),
+           ROUTE_RULES[rule], float(scale), width, router.shape[0], int(n_identity), int(groups), int(keep_groups), top, choice.data_ptr(), in_weight.data_ptr(),
            out_weight.data_ptr(), _ptr(identity_weight), n, dtype_code(x.dtype), _stream())
 
 
@@ -1402,13 +1419,14 @@ def _check_identity(identity_weight, x, n, who):
 
 
 def experts(hidden, act, x, choice, in_weight, out_weight, gate_of, up_of, down_of, inner_of, max_inner, pairs, ld_down=None,
-            assign=False, identity_weight=None):
+            assign=False, identity_weight=None, form=None, limit=0.0, shared_limit=0.0, alpha=0.0, n_experts=-1):
     """hidden[t] += sum over the token's ``pairs`` of out_weight * W_down[e] (silu(W_gate[e] x') * (W_up[e] x')),
     x' = in_weight * x[t] rounded to the activations' type; expert e's matrices are named by the
     int64 pointer tables ``gate_of``, ``up_of``, ``down_of`` and its inner size by ``inner_of`` (int32);
     the rows of every down matrix lie ``ld_down`` elements apart (None: ``max_inner``, for experts of
     one size that are stored each by itself).  ``gate_of`` None: experts without a gate matrix,
-    W_down[e] relu(W_up[e] x')^2.  ``act`` [T * pairs, max_inner] is scratch.  A pair whose choice is negative has no
+    W_down[e] relu(W_up[e] x')^2.  ``form`` "clamped_glu": between the products g' sigmoid(alpha g') (u' + 1) with
+    g' = min(g, limit) and u' = clamp(u, -limit, limit); expert ``n_experts`` (the shared one) has ``shared_limit``.  ``act`` [T * pairs, max_inner] is scratch.  A pair whose choice is negative has no
     expert; with ``identity_weight`` [T] identity_weight[t] * x[t] joins the sum.  ``assign``: ``hidden`` is set
     to the sum instead of added to."""
     _check(hidden, "experts.hidden", torch.float32, 2)
@@ -1422,25 +1440,27 @@ def experts(hidden, act, x, choice, in_weight, out_weight, gate_of, up_of, down_
     if hidden.shape != (n, width) or act.shape[0] < n * pairs or act.shape[1] < max_inner:
         raise KernelError("experts: sizes do not agree")
     _check_identity(identity_weight, x, n, "experts")
+    form = form or ("gated_silu" if gate_of is not None else "relu_squared")
     _experts(hidden.data_ptr(), hidden.stride(0), act.data_ptr(), act.stride(0), x.data_ptr(), x.stride(0), choice.data_ptr(),
              in_weight.data_ptr(), out_weight.data_ptr(), _ptr(gate_of), up_of.data_ptr(), down_of.data_ptr(),
              inner_of.data_ptr(), int(ld_down if ld_down is not None else max_inner), int(max_inner), width, int(pairs),
-             _ptr(identity_weight), n, int(bool(assign)), dtype_code(x.dtype), _stream())
+             _ptr(identity_weight), EXPERT_FORMS[form], float(limit), float(shared_limit), float(alpha), int(n_experts), n,
+             int(bool(assign)), dtype_code(x.dtype), _stream())
     return hidden
 
 
-def expert_combine(act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs, gated=True, hidden=None, x=None,
-                   identity_weight=None, assign=False):
+def expert_combine(act, gu, choice, in_weight, out_weight, n_experts, inner, top, pairs, form="gated_silu", hidden=None, x=None,
+                   identity_weight=None, assign=False, limit=0.0, shared_limit=0.0, alpha=0.0):
     """For the products over all experts at once: ``gu`` [T, 2 * total] holds every expert's gate and
     up results ([gates | ups], routed expert e in columns [e * inner, (e + 1) * inner), the shared
     expert behind them); act[t, c] = silu(s g) * (s u) * out_weight with s the token's input weight
-    for the column's expert, or 0 for an expert it did not choose.  act: [T, total].  ``gated`` false: ``gu`` [T, total]
-    holds the ups alone and act[t, c] = relu(s u)^2 * out_weight.  With ``identity_weight`` [T] the fp32 ``hidden``
+    for the column's expert, or 0 for an expert it did not choose.  act: [T, total].  ``form`` "relu_squared": ``gu`` [T, total]
+    holds the ups alone and act[t, c] = relu(s u)^2 * out_weight; "clamped_glu": see ``experts``.  With ``identity_weight`` [T] the fp32 ``hidden``
     [T, width] also gets identity_weight[t] * x[t] (``assign``: is set to it)."""
     _check(act, "expert_combine.act", gu.dtype, 2)
     _check(gu, "expert_combine.gu", None, 2)
     n, total = act.shape
-    if gu.shape != (n, (2 if gated else 1) * total) or total < n_experts * inner or (pairs == top and total != n_experts * inner):
+    if gu.shape != (n, (1 if form == "relu_squared" else 2) * total) or total < n_experts * inner or (pairs == top and total != n_experts * inner):
         raise KernelError("expert_combine: sizes do not agree")
     _check_identity(identity_weight, x, n, "expert_combine")
     width = 0
@@ -1451,7 +1471,7 @@ def expert_combine(act, gu, choice, in_weight, out_weight, n_experts, inner, top
         if hidden.shape != (n, width):
             raise KernelError("expert_combine: the stream and the tokens have another shape")
     _expert_combine(act.data_ptr(), act.stride(0), gu.data_ptr(), gu.stride(0), choice.data_ptr(), in_weight.data_ptr(),
-                    out_weight.data_ptr(), n_experts, inner, total, top, pairs, int(bool(gated)),
+                    out_weight.data_ptr(), n_experts, inner, total, top, pairs, EXPERT_FORMS[form], float(limit), float(shared_limit), float(alpha),
                     hidden.data_ptr() if width else None, hidden.stride(0) if width else 0, x.data_ptr() if width else None,
                     x.stride(0) if width else 0, _ptr(identity_weight), width, int(bool(assign)), n, dtype_code(gu.dtype),
                     _stream())
@@ -1670,3 +1690,87 @@ def softcap(x, cap):
         raise KernelError("softcap: the rows must be contiguous")
     _softcap(x.data_ptr(), float(cap), x.numel(), _stream())
     return x
+
+
+# ---- what a token's identity adds beyond its embedding row ---------------------------------------------------
+
+_pair_embed = Function("token", "mllm_token_pair_embed", [P, P, P, P, P, P, P, P, P, P, L, L, L, I, I, F, I, P])
+_token_gate = Function("token", "mllm_token_gate", [P, P, P, P, L, P, I, I, I, I, I, P])
+_token_gate_rows = Function("token", "mllm_token_gate_rows", [P, P, P, L, P, I, I, I, I, P])
+_add_normed_norm = Function("token", "mllm_token_add_normed_norm", [P, P, P, F, P, P, F, I, I, I, P])
+ROW_IN_SHARED_MEMORY = 47 * 1024 // 4        # entries of a 32-bit row that the kernels above keep in shared memory
+
+
+def pair_embed(out, token_ids, positions, token_item, item_slot, item_offset, item_count, table, pairs, state, buckets, mul_prev,
+               mul_cur, scale=1.0):
+    """out[t] = scale * table[id] + pairs[(previous id * mul_prev + id * mul_cur) mod buckets], or + pairs[buckets] for a
+    sequence's first token (position 0).  The id before an entry's first token of the step comes from ``state`` [slots]
+    (int32), where the entry's last id is then left."""
+    _check(out, "pair_embed.out", torch.float32, 2)
+    _check(table, "pair_embed.table", None, 2)
+    _check(pairs, "pair_embed.pairs", table.dtype, 2)
+    _check(state, "pair_embed.state", torch.int32, 1)
+    for name, t in (("token_ids", token_ids), ("positions", positions), ("token_item", token_item), ("item_slot", item_slot),
+                    ("item_offset", item_offset), ("item_count", item_count)):
+        _check(t, f"pair_embed.{name}", torch.int32, 1)
+    n, width = out.shape
+    if not (out.is_contiguous() and table.is_contiguous() and pairs.is_contiguous() and state.is_contiguous()):
+        raise KernelError("pair_embed: the output, the tables and the state must be contiguous")
+    if table.shape[1] != width or pairs.shape != (buckets + 1, width) or min(token_ids.shape[0], positions.shape[0], token_item.shape[0]) < n:
+        raise KernelError("pair_embed: sizes do not agree")
+    _pair_embed(out.data_ptr(), token_ids.data_ptr(), positions.data_ptr(), token_item.data_ptr(), item_slot.data_ptr(),
+                item_offset.data_ptr(), item_count.data_ptr(), table.data_ptr(), pairs.data_ptr(), state.data_ptr(), int(buckets),
+                int(mul_prev), int(mul_cur), n, width, float(scale), dtype_code(table.dtype), _stream())
+    return out
+
+
+def _check_side(side, token_ids, first, dim, n, who):
+    _check(side, f"{who}.side", None, 2)
+    _check(token_ids, f"{who}.token_ids", torch.int32, 1)
+    if not side.is_contiguous() or first < 0 or first + dim > side.shape[1] or token_ids.shape[0] < n:
+        raise KernelError(f"{who}: columns {first} .. {first + dim - 1} of a row per token")
+
+
+def token_gate(out, x, w, side, token_ids, first):
+    """out[t, j] = gelu_tanh(w[j] . x[t]) * side[token_ids[t], first + j]; ``x`` the fp32 stream [T, width], ``w`` [dim, width]."""
+    _check(out, "token_gate.out", side.dtype, 2)
+    _check(x, "token_gate.x", torch.float32, 2)
+    _check(w, "token_gate.w", side.dtype, 2)
+    n, dim = out.shape
+    width = x.shape[1]
+    _check_side(side, token_ids, first, dim, n, "token_gate")
+    if w.shape != (dim, width) or x.shape[0] < n or not (out.is_contiguous() and x.is_contiguous() and w.is_contiguous()):
+        raise KernelError("token_gate: sizes do not agree")
+    _token_gate(out.data_ptr(), x.data_ptr(), w.data_ptr(), side.data_ptr(), side.stride(0), token_ids.data_ptr(), int(first), dim, width,
+                n, dtype_code(side.dtype), _stream())
+    return out
+
+
+def token_gate_rows(out, z, side, token_ids, first):
+    """out[t, j] = gelu_tanh(z[t, j]) * side[token_ids[t], first + j]; ``z`` fp32 [T, dim]."""
+    _check(out, "token_gate_rows.out", side.dtype, 2)
+    _check(z, "token_gate_rows.z", torch.float32, 2)
+    n, dim = out.shape
+    _check_side(side, token_ids, first, dim, n, "token_gate_rows")
+    if z.shape != (n, dim) or not (out.is_contiguous() and z.is_contiguous()):
+        raise KernelError("token_gate_rows: sizes do not agree")
+    _token_gate_rows(out.data_ptr(), z.data_ptr(), side.data_ptr(), side.stride(0), token_ids.data_ptr(), int(first), dim, n,
+                     dtype_code(side.dtype), _stream())
+    return out
+
+
+def add_normed_norm(hidden, y, gain, eps, normed, next_gain, next_eps):
+    """hidden += y / sqrt(mean(y^2) + eps) * gain on the fp32 stream, and normed = hidden / sqrt(mean(hidden^2) + next_eps) *
+    next_gain of the rows as they then are, rounded to ``normed``'s element type."""
+    _check(hidden, "add_normed_norm.hidden", torch.float32, 2)
+    _check(y, "add_normed_norm.y", torch.float32, 2)
+    _check(normed, "add_normed_norm.normed", None, 2)
+    _check(gain, "add_normed_norm.gain", torch.float32, 1)
+    _check(next_gain, "add_normed_norm.next_gain", torch.float32, 1)
+    n, width = hidden.shape
+    if (y.shape != (n, width) or normed.shape != (n, width) or gain.shape[0] != width or next_gain.shape[0] != width
+            or not (hidden.is_contiguous() and y.is_contiguous() and normed.is_contiguous())):
+        raise KernelError("add_normed_norm: sizes do not agree")
+    _add_normed_norm(hidden.data_ptr(), y.data_ptr(), gain.data_ptr(), float(eps), normed.data_ptr(), next_gain.data_ptr(), float(next_eps),
+                     width, n, dtype_code(normed.dtype), _stream())
+    return hidden

@@ -290,19 +290,24 @@ class NormedAttention(Mixer):
     own, times one gain of the head's size that all heads share; eps inside the root.  Then the position
     encoding (``position``: a part with ``norm_rotate_store``) turns q and k, and the keys and values go to the
     pages.  ``score = q . k * scale``, with ``softcap`` ``cap * tanh(score / cap)``, over the keys at positions <= the
-    query's (of those the last ``window`` if given, and the first ``keep_first`` of the sequence); with ``sink`` the
+    query's (of those the last ``window`` if given, and the first ``keep_first`` of the sequence); ``distance_slopes`` (one
+    number per head) take slope[h] * (query's position - key's position) off the capped score; with ``sink`` the
     softmax's denominator also holds ``exp(sink[h])``, a learned number per head that has no key and no value, or, with
     ``sink="zero"``, exp(0) = 1 for every head; softmax and the weighted sum in
-    32-bit; query head h reads key/value head ``h // (heads / kv_heads)``; then ``W_o``.  ``own_kv=False``: the part
+    32-bit; query head h reads key/value head ``h // (heads / kv_heads)``.  ``gate``: entry by entry the
+    concatenated heads are multiplied by ``sigmoid(W_g x)`` (rows of the same stacked product); then ``W_o``.  ``position=None``:
+    nothing turns.  ``own_kv=False``: the part
     has no keys and values (no projections, taps or norm of them): it attends, with its own queries, over the
-    pages of the run entry named by ``RunEntry.cache_of``."""
+    pages of the run entry named by ``RunEntry.cache_of``; the entry whose pages others read keeps ``keep`` >= ``window``
+    positions (the widest window of all that read them; ``keep=0``: all positions, for a reader without a window)."""
 
     graph_safe = True
 
     def __init__(self, prefix, width: int, n_heads: int, n_kv_heads: int, key_size: int, value_size: int, score_scale: float,
-                 eps: float, position, norm: str | None = "whole", values: str = "projected", taps: int | None = None,
+                 eps: float, position=None, norm: str | None = "whole", values: str = "projected", taps: int | None = None,
                  softcap: float | None = None, window: int | None = None, sink: bool | str = False, own_kv: bool = True,
-                 keep_first: int = 0, bias: bool = False, names: dict | None = None):
+                 keep_first: int = 0, bias: bool = False, gate: bool = False, distance_slopes=None, keep: int | None = None,
+                 names: dict | None = None):
         super().__init__(prefix)
         self.width, self.n_heads, self.n_kv_heads = int(width), int(n_heads), int(n_kv_heads)
         self.dim, self.vdim, self.taps = int(key_size), int(value_size), int(taps) if taps is not None else 0
@@ -311,7 +316,13 @@ class NormedAttention(Mixer):
         self.window = int(window) if window else None
         if sink not in (False, True, "zero"):
             raise ValueError(f"{prefix}: a sink is learned (True), 'zero' or absent (False), got {sink!r}")
-        self.sink, self.own_kv, self.bias = sink, bool(own_kv), bool(bias)
+        self.sink, self.own_kv, self.bias, self.gate = sink, bool(own_kv), bool(bias), bool(gate)
+        self.distance_slopes = tuple(float(slope) for slope in distance_slopes) if distance_slopes is not None else None
+        if self.distance_slopes is not None and len(self.distance_slopes) != self.n_heads:
+            raise ValueError(f"{prefix}: {len(self.distance_slopes)} distance slopes for {self.n_heads} heads")
+        self.keep = self.window
+        if self.window and keep is not None:
+            self.keep = max(int(keep), self.window) if keep else None
         self.keep_first = int(keep_first) if self.window else 0        # (without a window every key is visible anyway)
         if self.keep_first < 0:
             raise ValueError(f"{prefix}: a negative number of first tokens cannot be kept")
@@ -326,10 +337,10 @@ class NormedAttention(Mixer):
         if self.taps < 0:
             raise ValueError(f"{prefix}: a convolution has at least one tap")
         self.norm, self.values = norm, values
-        self.position = build_part(position)
-        if not hasattr(self.position, "norm_rotate_store"):
+        self.position = build_part(position) if position is not None else None
+        if self.position is not None and not hasattr(self.position, "norm_rotate_store"):
             raise ValueError(f"{prefix}: the position encoding '{position.kind}' has no norm_rotate_store(ctx, cache, qkv, ...)")
-        self.names = dict(q="q", k="k", v="v", o="o", norm=".norm", taps=".conv", bias=".b", sink="sink")
+        self.names = dict(q="q", k="k", v="v", o="o", g="g", norm=".norm", taps=".conv", bias=".b", sink="sink")
         self.names.update(names or {})
         self.q_width, self.k_width, self.v_width = self.n_heads * self.dim, self.n_kv_heads * self.dim, self.n_kv_heads * self.vdim
         self.projections = [("q", self.q_width)]
@@ -338,10 +349,11 @@ class NormedAttention(Mixer):
             if values == "projected":
                 self.projections.append(("v", self.v_width))
         self.proj_width = sum(rows for _, rows in self.projections)
+        self.gate_width = self.n_heads * self.vdim if self.gate else 0
 
     def weight_specs(self):
         n = self.names
-        specs = list(self.position.weight_specs())
+        specs = list(self.position.weight_specs()) if self.position is not None else []
         for key, rows in self.projections:
             specs.append(WeightSpec(self.full_name(n[key]), (rows, self.width)))
             if self.bias:
@@ -351,6 +363,8 @@ class NormedAttention(Mixer):
             if self.norm is not None and key != "v":
                 specs.append(WeightSpec(self.full_name(n[key] + n["norm"]), (rows if self.norm == "whole" else self.dim,),
                                         role="vector", init="gain"))
+        if self.gate:
+            specs.append(WeightSpec(self.full_name(n["g"]), (self.gate_width, self.width)))
         if self.sink is True:
             specs.append(WeightSpec(self.full_name(n["sink"]), (self.n_heads,), role="vector", init="shift"))
         specs.append(WeightSpec(self.full_name(n["o"]), (self.width, self.n_heads * self.vdim), init="residual_matrix"))
@@ -358,7 +372,7 @@ class NormedAttention(Mixer):
 
     def cache_need(self):
         # (an entry that reads another's pages gets them under the same name, "kv")
-        need = {"kv": PagedKV(self.n_kv_heads, self.dim, self.window, value_size=self.vdim, keep_first=self.keep_first)}
+        need = {"kv": PagedKV(self.n_kv_heads, self.dim, self.keep, value_size=self.vdim, keep_first=self.keep_first)}
         if self.taps > 1:
             need["taps"] = FixedState((self.taps - 1, self.proj_width), "float32")
         return need
@@ -366,11 +380,20 @@ class NormedAttention(Mixer):
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
         n = self.names
-        self.position.bind({w.name: tensors[w.name] for w in self.position.weight_specs() if w.name in tensors}, runtime)
+        if self.position is not None:
+            self.position.bind({w.name: tensors[w.name] for w in self.position.weight_specs() if w.name in tensors}, runtime)
         keys = [key for key, _ in self.projections]
-        self.stacked = torch.cat([self.w(n[key]) for key in keys]).contiguous()
+        # (the gate's rows stand behind the projections')
+        self.stacked = torch.cat([self.w(n[key]) for key in keys] + ([self.w(n["g"])] if self.gate else [])).contiguous()
         self.stacked_taps = torch.cat([self.w(n[key] + n["taps"]) for key in keys]).contiguous() if self.taps >= 1 else None
-        self.stacked_bias = torch.cat([self.w(n[key] + n["bias"]) for key in keys]).contiguous() if self.bias else None
+        self.stacked_bias = None
+        if self.bias:
+            none = [torch.zeros(self.gate_width, dtype=torch.float32, device=self.stacked.device)] if self.gate else []
+            self.stacked_bias = torch.cat([self.w(n[key] + n["bias"]) for key in keys] + none).contiguous()
+        self.slopes = None
+        if self.distance_slopes is not None:
+            self.slopes = torch.tensor(self.distance_slopes, dtype=torch.float32, device=self.stacked.device)
+        self._no_turns = torch.zeros(1, dtype=torch.float64, device=self.stacked.device)
         self.sinks = None
         if self.sink is True:
             self.sinks = self.w(n["sink"])
@@ -388,7 +411,7 @@ class NormedAttention(Mixer):
             raise RuntimeError(f"{self.prefix}: a part {'with' if self.own_kv else 'without'} keys and values of its own got pages "
                                f"it may {'not ' if self.own_kv else ''}store into (RunEntry.cache_of)")
         # projections, taps, norm and rotation in 32-bit: the queries and the cache are rounded once
-        projected = ctx.buffer("qkv_32", (n, self.proj_width), torch.float32)
+        projected = ctx.buffer("qkv_32", (n, self.proj_width + self.gate_width), torch.float32)
         k.linear(ctx, projected, x, self.stacked, self.stacked_bias)
         taps = None
         if self.taps >= 1:
@@ -396,11 +419,16 @@ class NormedAttention(Mixer):
         q = ctx.buffer("q", (n, self.q_width), ctx.act_dtype)
         k_off = self.q_width
         v_off = k_off + self.k_width if self.values == "projected" else k_off
-        self.position.norm_rotate_store(ctx, pages, projected, q, k_off, v_off, self.n_heads, self.n_kv_heads, self.dim, self.vdim,
-                                        self.q_gain, self.k_gain, self.norm, self.eps, taps)
+        if self.position is not None:
+            self.position.norm_rotate_store(ctx, pages, projected, q, k_off, v_off, self.n_heads, self.n_kv_heads, self.dim, self.vdim,
+                                            self.q_gain, self.k_gain, self.norm, self.eps, taps)
+        else:
+            k.norm_rotary_store(ctx, pages, projected, q, k_off, v_off, self.n_heads, self.n_kv_heads, self.dim, self.vdim,
+                                self.q_gain, self.k_gain, self.norm, self.eps, 0, "interleaved", self._no_turns, taps)
         mixed = ctx.buffer("attn_out", (n, self.n_heads * self.vdim), ctx.act_dtype)
         k.capped_attention(ctx, mixed, q, pages, self.n_heads, self.n_kv_heads, self.dim, self.vdim, self.score_scale,
-                           self.softcap, self.window or 0, sink=self.sinks, keep=self.keep_first)
+                           self.softcap, self.window or 0, sink=self.sinks, keep=self.keep_first, slopes=self.slopes,
+                           gate=projected[:, self.proj_width:] if self.gate else None, gate_wide=self.gate)
         return mixed
 
     def compute(self, ctx, x, cache):

@@ -28,7 +28,8 @@ residual stream [T, width]; "act" tensors have the engine's element type):
     for encodings that act on the embedded tokens; ``additive_table()`` may
     return the table so that the embedding gather fuses the sum.  Encodings
     that act inside a mixer are given to that mixer as a parameter instead.
-``Embedding.forward(ctx, position=None) -> hidden``
+``Embedding.forward(ctx, position=None, cache=None) -> hidden``
+    ``cache_need()`` as for a mixer, for an embedding that keeps something per request (its view is ``cache``).
 ``Head.forward(ctx, x) -> fp32 logits [R, vocab]``
 ``Arrangement.run(ctx, parts, hidden, cache)``
     wire one layer's parts (by role) around the residual stream.
@@ -103,7 +104,10 @@ class PositionEncoding(Part):
 
 
 class Embedding(Part):
-    def forward(self, ctx, position=None):
+    def cache_need(self):
+        return NoCache()
+
+    def forward(self, ctx, position=None, cache=None):
         raise NotImplementedError
 
 
@@ -116,6 +120,8 @@ class Arrangement:
     """How the parts of one layer are wired; ``roles`` names the parts it needs."""
 
     roles: tuple = ()
+    first_norm: str | None = None      # the role whose norm is the first thing that reads the stream, if that is so: a pass
+                                       # that changes the stream last may apply it (``ctx.normed_ahead``)
 
     def run(self, ctx, parts: dict, hidden, cache) -> None:
         raise NotImplementedError

@@ -2,7 +2,8 @@
 
 "pre_norm" is the reference's block (engine/src/transformer_block.c:49-71):
 ``r = x + mixer(norm_1(x))``, then ``out = r + feed_forward(norm_2(r))``.  The
-residual stream stays 32-bit; mixers and feed-forwards add into it in place.
+residual stream stays 32-bit; mixers and feed-forwards add into it in place.  A layer may have a "token_side" part that
+then adds what the token's identity gives this layer; its pass may also have applied the next layer's norm_1.
 
 "sandwich_norm" norms every sublayer on both sides:
 ``x <- x + norm_1b(mixer(filter(norm_1(x))))``, then, if the layer has a feed-forward,
@@ -38,18 +39,25 @@ def _defer(norm, consumer) -> dict:
 
 class PreNorm(Arrangement):
     roles = ("norm_1", "mixer")
-    optional_roles = ("norm_2", "feed_forward")      # a layer may have no feed-forward
+    optional_roles = ("norm_2", "feed_forward", "token_side")      # a layer may have no feed-forward
+    first_norm = "norm_1"
 
     def run(self, ctx, parts, hidden, cache):
         # A part that states ``accepts_deferred_norm`` may get its input norm unevaluated
         # (to fuse it into its first product); any other part gets a tensor.
-        x = parts["norm_1"].forward(ctx, hidden, tag="norm_1", **_defer(parts["norm_1"], parts["mixer"]))
+        ahead, ctx.normed_ahead = getattr(ctx, "normed_ahead", None), None
+        if ahead is not None and ahead[0] is parts["norm_1"]:
+            x = ahead[1]                             # (the pass that changed the stream last applied this norm)
+        else:
+            x = parts["norm_1"].forward(ctx, hidden, tag="norm_1", **_defer(parts["norm_1"], parts["mixer"]))
         if getattr(cache, "kind", "none") == "composite":
             cache = cache.sub("mixer")               # a mixer that keeps several things gets them by its own names
         parts["mixer"].forward(ctx, x, hidden, cache)
         if "feed_forward" in parts:
             x = parts["norm_2"].forward(ctx, hidden, tag="norm_2", **_defer(parts["norm_2"], parts["feed_forward"]))
             parts["feed_forward"].forward(ctx, x, hidden)
+        if "token_side" in parts:
+            parts["token_side"].forward(ctx, hidden)
 
 
 class SandwichNorm(Arrangement):

@@ -14,7 +14,7 @@ from __future__ import annotations
 import torch
 
 from .base import Embedding, Head, PositionEncoding, register_part
-from .spec import WeightSpec
+from .spec import FixedState, WeightSpec
 
 
 class TokenEmbedding(Embedding):
@@ -26,11 +26,38 @@ class TokenEmbedding(Embedding):
     def weight_specs(self):
         return [WeightSpec(self.full_name(self.name), (self.vocab_size, self.width), role="table", init="table")]
 
-    def forward(self, ctx, position=None):
+    def forward(self, ctx, position=None, cache=None):
         hidden = ctx.buffer("hidden", (ctx.n_tokens, self.width), torch.float32)
         table = position.additive_table() if position is not None else None
         ctx.kernels.embed(hidden, ctx.token_ids, ctx.positions, self.w(self.name), table, self.scale)
         if position is not None and table is None:
+            position.add_to_hidden(ctx, hidden)
+        return hidden
+
+
+class PairedTokenEmbedding(TokenEmbedding):
+    """The token's row plus a row for the pair of it and the token before it: row
+    ``(previous * mul_prev + token * mul_cur) mod buckets`` of a table of ``buckets + 1`` rows, the last of which is for a
+    sequence's first token.  A request's last token is its state."""
+
+    def __init__(self, prefix, vocab_size: int, width: int, buckets: int, mul_prev: int, mul_cur: int, name: str = "wte.weight",
+                 pair_name: str = "bigram", scale: float = 1.0):
+        super().__init__(prefix, vocab_size, width, name, scale)
+        self.buckets, self.mul_prev, self.mul_cur, self.pair_name = int(buckets), int(mul_prev), int(mul_cur), pair_name
+        if self.buckets < 1 or min(self.mul_prev, self.mul_cur) < 0:
+            raise ValueError(f"{self.full_name(pair_name)}: a positive number of buckets and factors that are not negative")
+
+    def weight_specs(self):
+        return super().weight_specs() + [WeightSpec(self.full_name(self.pair_name), (self.buckets + 1, self.width), role="table", init="table")]
+
+    def cache_need(self):
+        return FixedState((1,), "int32")
+
+    def forward(self, ctx, position=None, cache=None):
+        hidden = ctx.buffer("hidden", (ctx.n_tokens, self.width), torch.float32)
+        ctx.kernels.pair_embed(ctx, hidden, self.w(self.name), self.w(self.pair_name), cache.state.view(-1), self.buckets, self.mul_prev,
+                               self.mul_cur, self.scale)
+        if position is not None:
             position.add_to_hidden(ctx, hidden)
         return hidden
 
@@ -78,5 +105,6 @@ class LinearHead(Head):
 
 
 register_part("token_embedding", TokenEmbedding)
+register_part("paired_token_embedding", PairedTokenEmbedding)
 register_part("learned_positions", LearnedPositions)
 register_part("linear_head", LinearHead)

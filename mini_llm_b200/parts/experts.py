@@ -20,6 +20,12 @@ ones' sum (+ 1e-20), times ``router_scale``.  The router may have ``n_identity``
 with matrices, the last ones: experts whose output is the token itself (times the weight).  ``form="relu_squared"``:
 experts without a gate, ``W_down relu(W_up u)^2``.
 
+``weights="sigmoid"``: scores ``s = sigmoid(z)``; ``s`` plus the correction ranks the outputs, the chosen experts' outputs are
+weighed by ``s`` itself (not renormalized), times ``router_scale``.  ``groups=(count, keep)``: the outputs form ``count`` equal
+runs of neighbours, a run counts the sum of its two largest ranking scores, and only the ``keep`` best runs' experts can be
+chosen.  ``form="clamped_glu"``: experts ``W_down (g sigmoid(alpha g) (v + 1))`` with ``g = min(W_gate u, limit)`` and
+``v = clamp(W_up u, -limit, limit)``; the shared expert has a limit of its own.
+
 Experts are named by tables of pointers and inner sizes, so the shared expert goes through the
 kernels as one more chosen expert with input weight 1 and its gate as the output weight.  A step
 of few tokens runs pair by pair (token, chosen expert) and reads only the chosen experts'
@@ -39,20 +45,21 @@ from .spec import WeightSpec
 class RoutedExperts(FeedForward):
     graph_safe = True
 
-    WEIGHTS = ("sigmoid_on_input", "softmax_of_chosen", "softmax_of_all")
-    FORMS = ("gated_silu", "relu_squared")
+    WEIGHTS = ("sigmoid_on_input", "softmax_of_chosen", "softmax_of_all", "sigmoid")
+    FORMS = ("gated_silu", "relu_squared", "clamped_glu")
 
     def __init__(self, prefix, width: int, n_experts: int, top: int, expert_inner: int, shared_inner: int | None = None,
                  names: dict | None = None, weights: str = "sigmoid_on_input", router_bias: bool = False,
                  shared_gate: bool = True, form: str = "gated_silu", n_identity: int = 0, correction: bool = False,
-                 router_scale: float = 1.0):
+                 router_scale: float = 1.0, groups=None, limit: float | None = None, shared_limit: float | None = None,
+                 alpha: float = 1.702):
         super().__init__(prefix)
         if weights not in self.WEIGHTS:
             raise ValueError(f"{prefix}: unknown rule for the experts' weights '{weights}' (known: {', '.join(self.WEIGHTS)})")
         self.weights_rule, self.router_bias, self.shared_gate = weights, bool(router_bias), bool(shared_gate)
         if form not in self.FORMS:
             raise ValueError(f"{prefix}: unknown form of an expert '{form}' (known: {', '.join(self.FORMS)})")
-        self.gated, self.n_identity, self.correction = form == "gated_silu", int(n_identity), bool(correction)
+        self.form, self.gated, self.n_identity, self.correction = form, form != "relu_squared", int(n_identity), bool(correction)
         self.router_scale = float(router_scale)
         self.width, self.n_experts, self.top, self.inner = int(width), int(n_experts), int(top), int(expert_inner)
         self.shared_inner = int(shared_inner) if shared_inner else None
@@ -60,9 +67,18 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"{prefix}: {self.n_experts} experts and {self.n_identity} identity experts")
         if self.n_identity and weights == "sigmoid_on_input":
             raise ValueError(f"{prefix}: identity experts need weights on the experts' outputs")
-        if (self.correction or self.router_scale != 1.0) and weights != "softmax_of_all":
-            raise ValueError(f"{prefix}: a correction and a scale belong to the softmax over all outputs")
+        if (self.correction or self.router_scale != 1.0) and weights not in ("softmax_of_all", "sigmoid"):
+            raise ValueError(f"{prefix}: a correction and a scale belong to the softmax over all outputs and to sigmoid scores")
         self.outputs = self.n_experts + self.n_identity
+        self.groups, self.keep_groups = (int(groups[0]), int(groups[1])) if groups else (0, 0)
+        if groups and (self.groups < 1 or self.outputs % self.groups or not 1 <= self.keep_groups <= self.groups
+                       or self.keep_groups * (self.outputs // self.groups) < top):
+            raise ValueError(f"{prefix}: {self.outputs} experts in {self.groups} equal groups, {self.keep_groups} of them kept, must leave {top} to choose")
+        self.form_constants = {"form": form}
+        if form == "clamped_glu":
+            if limit is None or (shared_inner and shared_limit is None):
+                raise ValueError(f"{prefix}: clamped experts need their limit")
+            self.form_constants.update(limit=float(limit), shared_limit=float(shared_limit or 0.0), alpha=float(alpha))
         if not 1 <= self.top <= self.outputs:
             raise ValueError(f"{prefix}: every token takes between 1 and {self.outputs} experts, got {self.top}")
         if self.inner <= 0:
@@ -139,19 +155,20 @@ class RoutedExperts(FeedForward):
                 choice, in_weight, out_weight, bias=self.w(self.names["router_bias"]) if self.router_bias else None,
                 rule=self.weights_rule, shared_plain=bool(self.shared_inner) and not gated,
                 correction=self.w(self.names["correction"]) if self.correction else None, n_identity=self.n_identity,
-                scale=self.router_scale, identity_weight=identity)
+                scale=self.router_scale, identity_weight=identity, groups=self.groups, keep_groups=self.keep_groups)
         if k.experts_at_once(n, x, self.up_matrix, self.down_matrix):
             gu = ctx.buffer("expert_gate_up", (n, len(self._halves) * self.total), ctx.act_dtype)
             k.linear(ctx, gu, x, self.up_matrix)
             act = ctx.buffer("expert_act_all", (n, self.total), ctx.act_dtype)
             # (the identity experts' part goes onto the stream ahead of the product, which then adds)
             k.expert_combine(act, gu, choice, in_weight, out_weight, self.n_experts, self.inner, self.top, self.pairs,
-                             gated=self.gated, hidden=hidden, x=x, identity_weight=identity, assign=assign)
+                             **self.form_constants, hidden=hidden, x=x, identity_weight=identity, assign=assign)
             k.linear(ctx, hidden, act, self.down_matrix, None, epilogue="store" if assign and identity is None else "add")
             return
         act = ctx.buffer("expert_act", (n * self.pairs, self.max_inner), ctx.act_dtype)
         k.experts(hidden, act, x, choice, in_weight, out_weight, self.gate_of, self.up_of, self.down_of, self.inner_of,
-                  self.max_inner, self.pairs, ld_down=self.total, assign=assign, identity_weight=identity)
+                  self.max_inner, self.pairs, ld_down=self.total, assign=assign, identity_weight=identity,
+                  n_experts=self.n_experts, **self.form_constants)
 
     def compute(self, ctx, x):
         out = ctx.buffer("mlp_out", (x.shape[0], self.width), torch.float32)

@@ -15,13 +15,16 @@ and a single decoded token take the same path, and no key or value per head is e
 
 Rotary positions: among the first ``rotary_dims`` entries of the rotated part, pair i turns by
 ``position * base^(-2i/rotary_dims)``; ``rotary_layout`` says which entries form pair i: 2i and 2i+1
-("interleaved") or i and i + rotary_dims/2 ("half").
+("interleaved") or i and i + rotary_dims/2 ("half").  ``rotary_scaling`` blends the frequencies and multiplies cosine and
+sine of both the queries and the shared key part (YaRN, see ``parts.rotary``); the unrotated part is not scaled.
 
 Options: ``window``: a query sees only the last ``window`` positions (itself included); the cache then
 keeps ``keep`` >= ``window`` positions (``keep``: the widest window of all entries that read these
 rows).  ``query_rank``: the queries go through a latent of their own, ``q = W_uq rms(W_dq x) * g_q``.
 ``own_rows=False``: the part has no down projection and stores nothing; it attends over the rows that
 another run entry stores (``RunEntry.cache_of``), with its own expansions, queries and mask.
+``gate``: head h's result is multiplied by ``sigmoid(w_g[h] . x)``, one number per token and head read off the same input;
+its rows stand behind the down projection's in one product, and it opens the weighted sum of latents, ahead of U_v.
 """
 
 from __future__ import annotations
@@ -29,6 +32,7 @@ from __future__ import annotations
 import torch
 
 from .base import Mixer, register_part
+from .rotary import rotary_frequencies
 from .spec import PagedKV, WeightSpec
 
 
@@ -42,7 +46,7 @@ class LatentAttention(Mixer):
                  key_up_name: str = "uk", value_up_name: str = "uv", out_name: str = "o", window: int | None = None,
                  keep: int | None = None, rotary_layout: str = "interleaved", query_rank: int | None = None,
                  query_down_name: str = "dq", query_norm_name: str = "dq.norm", query_up_name: str = "uq",
-                 own_rows: bool = True):
+                 own_rows: bool = True, rotary_scaling=None, gate: bool = False, gate_name: str = "g"):
         super().__init__(prefix)
         self.width, self.n_heads = int(width), int(n_heads)
         self.dim, self.rot, self.vdim, self.rank = int(head_size), int(rotated_size), int(value_size), int(latent_size)
@@ -54,7 +58,7 @@ class LatentAttention(Mixer):
         if min(self.n_heads, self.dim, self.vdim, self.rank) <= 0:
             raise ValueError(f"{prefix}: heads, head size, value size and latent size must be positive")
         self.names = dict(q=q_name, down=down_name, norm=latent_norm_name, uk=key_up_name, uv=value_up_name, o=out_name,
-                          dq=query_down_name, dq_norm=query_norm_name, uq=query_up_name)
+                          dq=query_down_name, dq_norm=query_norm_name, uq=query_up_name, g=gate_name)
         self.row = self.rank + self.rot
         self.window = int(window) if window else None
         self.keep = max(int(keep), self.window) if keep and self.window else self.window
@@ -62,7 +66,11 @@ class LatentAttention(Mixer):
             raise ValueError(f"{prefix}: unknown layout of the rotated pairs '{rotary_layout}' (known: half, interleaved)")
         self.rotary_layout = rotary_layout
         self.query_rank = int(query_rank) if query_rank else None
-        self.own_rows = bool(own_rows)
+        self.own_rows, self.gate = bool(own_rows), bool(gate)
+        self.frequencies, self.amplitude = [], 1.0
+        if self.rotary_dims:
+            self.frequencies, self.amplitude = rotary_frequencies(self.rotary_base, self.rotary_dims,
+                                                                  dict(rotary_scaling) if rotary_scaling else None)
 
     def weight_specs(self):
         n, h = self.names, self.n_heads
@@ -75,6 +83,8 @@ class LatentAttention(Mixer):
         if self.own_rows:
             specs += [WeightSpec(self.full_name(n["down"]), (self.row, self.width)),
                       WeightSpec(self.full_name(n["norm"]), (self.rank,), role="vector", init="gain")]
+        if self.gate:
+            specs.append(WeightSpec(self.full_name(n["g"]), (h, self.width)))
         return specs + [
             WeightSpec(self.full_name(n["uk"]), (h * self.dim, self.rank)),
             WeightSpec(self.full_name(n["uv"]), (h * self.vdim, self.rank)),
@@ -91,11 +101,15 @@ class LatentAttention(Mixer):
         # per head, [rank, dim]: the key expansion as the product's weight on the query's side
         self.key_up_t = uk.view(h, self.dim, self.rank).transpose(1, 2).contiguous()
         self.value_up = self.w(self.names["uv"]).view(h, self.vdim, self.rank)
-        half = self.rotary_dims // 2
-        exponent = -2.0 * torch.arange(half, dtype=torch.float64) / max(self.rotary_dims, 1)
-        self.inv_freq = (torch.tensor(self.rotary_base, dtype=torch.float64) ** exponent).to(uk.device)
-        if half == 0:
-            self.inv_freq = torch.zeros(1, dtype=torch.float64, device=uk.device)
+        self.inv_freq = torch.tensor(self.frequencies or [0.0], dtype=torch.float64, device=uk.device)
+        # what leaves its product in 32-bit: the down projection, and behind it the gate (by itself padded to the least a tile takes)
+        rows = ([self.w(self.names["down"])] if self.own_rows else []) + ([self.w(self.names["g"])] if self.gate else [])
+        self.thin = None
+        if rows:
+            short = 16 - sum(one.shape[0] for one in rows)
+            if short > 0:
+                rows.append(torch.zeros((short, self.width), dtype=uk.dtype, device=uk.device))
+            self.thin = torch.cat(rows).contiguous() if len(rows) > 1 else rows[0]
         self._no_gain = torch.ones(self.rank, dtype=torch.float32, device=uk.device)
 
     def compute(self, ctx, x, cache):
@@ -113,16 +127,22 @@ class LatentAttention(Mixer):
             k.linear(ctx, q, normed, self.w(names["uq"]))
         else:
             k.linear(ctx, q, x, self.w(names["q"]))
-        down = None
-        if self.own_rows:
-            down = ctx.buffer("latent_down", (n, self.row), torch.float32)
-            k.linear(ctx, down, x, self.w(names["down"]))
+        down = gate = None
+        if self.thin is not None:
+            thin = ctx.buffer("latent_down", (n, self.thin.shape[0]), torch.float32)
+            k.linear(ctx, thin, x, self.thin)
+            down = thin[:, :self.row] if self.own_rows else None
+            if self.gate:
+                first = self.row if self.own_rows else 0
+                gate = thin[:, first:first + h]
         q_eff = ctx.buffer("latent_q_eff", (n, h * self.row), torch.float32)
         k.latent_prepare(ctx, cache, q_eff, down, q, self.w(names["norm"]) if self.own_rows else self._no_gain, self.inv_freq,
-                         self.rank, self.rot, self.rotary_dims, h, self.dim, self.eps, layout=self.rotary_layout)
+                         self.rank, self.rot, self.rotary_dims, h, self.dim, self.eps, layout=self.rotary_layout,
+                         amplitude=self.amplitude)
         k.head_linear(ctx, q_eff, q, self.key_up_t, h, self.dim + self.rot, self.row)
         mixed_latent = ctx.buffer("latent_mixed", (n, h * self.rank), k.latent_mixed_dtype(cache, self.rank, self.rot))
-        k.latent_attention(ctx, mixed_latent, q_eff, cache, h, self.rank, self.rot, self.score_scale, window=self.window or 0)
+        k.latent_attention(ctx, mixed_latent, q_eff, cache, h, self.rank, self.rot, self.score_scale, window=self.window or 0,
+                           gate=gate)
         mixed = ctx.buffer("attn_out", (n, h * self.vdim), ctx.act_dtype)
         k.head_linear(ctx, mixed, mixed_latent, self.value_up, h, self.rank, self.vdim)
         out = ctx.buffer("mixer_out", (n, self.width), torch.float32)

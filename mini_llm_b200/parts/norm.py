@@ -7,7 +7,8 @@ consecutive pieces, each divided by ``sqrt(mean(piece^2) + eps)``, and the whole
 gain vector; ``groups=1`` is the plain RMS norm.  Besides the interface of every norm it can norm
 the residual stream in place and add a normed sublayer result onto it, which is what an
 arrangement with norms on both sides of a sublayer needs.  With ``unit_offset`` the stored weight lies
-around zero and the gain is ``1 + weight`` (added once, in 32-bit, when the weights arrive)."""
+around zero and the gain is ``1 + weight`` (added once, in 32-bit, when the weights arrive); ``scale`` multiplies the gain in
+the same way (a constant on logits, for instance, costs nothing on the norm ahead of their product)."""
 
 from __future__ import annotations
 
@@ -47,10 +48,11 @@ class GroupedRmsNorm(Norm):
     graph_safe = True
     can_defer = True
 
-    def __init__(self, prefix, width: int, eps: float, groups: int = 1, name: str = "weight", unit_offset: bool = False):
+    def __init__(self, prefix, width: int, eps: float, groups: int = 1, name: str = "weight", unit_offset: bool = False,
+                 scale: float = 1.0):
         super().__init__(prefix)
         self.width, self.eps, self.groups, self.name = int(width), float(eps), int(groups), name
-        self.unit_offset = bool(unit_offset)
+        self.unit_offset, self.scale = bool(unit_offset), float(scale)
         if self.groups <= 0 or self.width % self.groups != 0:
             raise ValueError(f"{self.full_name(name)}: a width of {self.width} does not split into {self.groups} equal groups")
 
@@ -61,6 +63,9 @@ class GroupedRmsNorm(Norm):
         if self.unit_offset:
             name = self.full_name(self.name)
             tensors = {**tensors, name: tensors[name] + 1.0}
+        if self.scale != 1.0:
+            name = self.full_name(self.name)
+            tensors = {**tensors, name: tensors[name] * self.scale}
         super().bind(tensors, runtime)
 
     def forward(self, ctx, x, rows=None, tag="norm", defer=False):
@@ -78,6 +83,11 @@ class GroupedRmsNorm(Norm):
         """The fp32 stream itself is normed (after an embedding, for instance)."""
         ctx.kernels.grouped_rms_norm(hidden, hidden, self.w(self.name), self.groups, self.eps)
         return hidden
+
+    @property
+    def whole_row(self) -> bool:
+        """Whether a pass over the stream can apply this norm itself: one root mean square over the whole row, one gain."""
+        return self.groups == 1
 
     def add_normed(self, ctx, hidden, y, rounded=None):
         """hidden += norm(y): a sublayer's fp32 result is normed on its way onto the stream.  ``rounded``: the

@@ -501,7 +501,7 @@ def test_router_with_corrections_and_identity_experts(experts, identity, top):
         np.testing.assert_allclose(hidden.cpu().numpy(), expected + (0.0 if assign else before), atol=3e-5)
         hidden, gu = dev(before), dev(x) @ up_matrix.T
         combined = torch.full((n, experts * inner), float("nan"), device="cuda")
-        ops.expert_combine(combined, gu.contiguous(), choice, in_weight, out_weight, experts, inner, top, top, gated=False, hidden=hidden,
+        ops.expert_combine(combined, gu.contiguous(), choice, in_weight, out_weight, experts, inner, top, top, form="relu_squared", hidden=hidden,
                            x=dev(x), identity_weight=passed if identity else None, assign=assign)
         if assign and not identity:
             hidden.zero_()
