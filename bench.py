@@ -64,7 +64,7 @@ def parse_args():
     parser.add_argument("--kernels", action="store_true",
                         help="time single kernels (matrix products at forced tile widths, prompt attention) back to "
                              "back in a replayed graph and print one line each: the tables of profiles/ come from this")
-    parser.add_argument("--compare", default=None, choices=("fuvolix", "sumozen", "lipulorn", "deluvik", "nufavik"),
+    parser.add_argument("--compare", default=None, choices=("fuvolix", "sumozen", "lipulorn", "deluvik", "nufavik", "kerepel"),
                         help="fuvolix: prefill and decode of Fuvolix stacks at sizes of real layers (random weights), beside "
                              "GPT-2 of equal width, depth and inner size, and their mixers' kernels alone; sumozen: Sumozen "
                              "stacks beside Fuvolix stacks of equal width, depth and inner size, and its kernels alone; "
@@ -73,6 +73,8 @@ def parse_args():
                              "Sumozen stacks of equal width, depth and experts, and its kernels alone beside Sumozen's like kernels; "
                              "nufavik: Nufavik stacks beside Deluvik stacks of equal width, depth, heads and experts, and its kernels "
                              "alone beside Deluvik's like kernels; "
+                             "kerepel: Kerepel stacks beside Deluvik stacks of equal width, depth, heads and feed-forward weights, and its "
+                             "kernels alone beside the closest designs' like kernels; "
                              "one line each")
     parser.add_argument("--tokens-out", default=None,
                         help="(--impl reference) write the greedy tokens of the fixed check workload to this file "
@@ -1704,6 +1706,276 @@ def run_compare_nufavik(args):
     return 0
 
 
+KEREPEL_SIZES = {
+    "768 wide": {"width": 768, "layers": 12, "ff": 3072, "side": 64, "taps": 4, "window": 512,
+                 "attention": {"heads": 12, "kv_heads": 4, "dim": 64, "vdim": 64},
+                 "latent": {"heads": 12, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256},
+                 "moe": {"experts": 16, "groups": 4, "keep": 2, "top": 2, "ff": 512, "shared": 512}},
+    "1,024 wide": {"width": 1024, "layers": 24, "ff": 4096, "side": 128, "taps": 4, "window": 512,
+                   "attention": {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 96},
+                   "latent": {"heads": 16, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 512},
+                   "moe": {"experts": 16, "groups": 4, "keep": 2, "top": 2, "ff": 512, "shared": 512}},
+    "2,048 wide": {"width": 2048, "layers": 12, "ff": 6144, "side": 256, "taps": 4, "window": 512,
+                   "attention": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128},
+                   "latent": {"heads": 16, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512},
+                   "moe": {"experts": 16, "groups": 4, "keep": 2, "top": 4, "ff": 1024, "shared": 1024}},
+}
+
+
+def kerepel_config(size: dict, vocab: int) -> dict:
+    att, lat, moe = size["attention"], size["latent"], size["moe"]
+    dense = {"kind": "dense", "ff": size["ff"]}
+    routed = {"kind": "moe", "router": {"experts": moe["experts"], "top": moe["top"], "groups": {"count": moe["groups"], "keep": moe["keep"]}},
+              "expert": {"ff": moe["ff"], "limit": 7.0}, "shared": {"ff": moe["shared"], "limit": 7.0}}
+    latent = dict(lat, scale=(lat["dim"] + lat["rot_dim"]) ** -0.5,
+                  rot={"base": 10000.0, "dims": lat["rot_dim"], "scaling": {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}})
+    windowed = dict(att, conv=size["taps"], scale=att["dim"] ** -0.5, softcap=50.0, mask={"size": size["window"]})
+    layers = []
+    while len(layers) < size["layers"]:
+        layers += [{"type": "latent_attention", "mixer": latent, "mlp": dense}, {"type": "attention", "mixer": windowed, "mlp": routed},
+                   {"type": "attention", "mixer": dict(windowed, kv_from=len(layers) + 1), "mlp": dense}]
+    return {"architecture": "Kerepel", "vocab": vocab, "width": size["width"], "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+            "embedding": {"bigram": {"buckets": 32749, "mul_prev": 10007, "mul_cur": 31}}, "token_side": {"dim": size["side"]},
+            "layers": layers[:size["layers"]]}
+
+
+def kerepel_like_config(size: dict, vocab: int) -> dict:
+    """Deluvik of equal width, depth, heads and feed-forward weights: attention over all keys where Kerepel has the latent."""
+    att, lat, moe = size["attention"], size["latent"], size["moe"]
+    dense = {"kind": "dense", "ff": size["ff"] * 2 // 3}                     # (three matrices, not two)
+    routed = {"kind": "moe", "router": {"experts": moe["experts"], "top": moe["top"]}, "expert": {"ff": moe["ff"]},
+              "shared": {"ff": moe["shared"]}}
+    rot = {"base": 10000.0, "dims": att["dim"]}
+    windowed = dict(att, conv=size["taps"], scale=att["dim"] ** -0.5, softcap=50.0, rot=rot, mask={"size": size["window"]})
+    full = dict(att, conv=size["taps"], scale=att["dim"] ** -0.5, softcap=50.0, rot=rot, heads=lat["heads"])
+    layers = []
+    while len(layers) < size["layers"]:
+        layers += [{"type": "attention_2", "mixer": full, "mlp": dense}, {"type": "attention_2", "mixer": windowed, "mlp": routed},
+                   {"type": "attention_2", "mixer": dict(windowed, kv_from=len(layers) + 1), "mlp": dense}]
+    return {"architecture": "Deluvik", "vocab": vocab, "width": size["width"], "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": layers[:size["layers"]]}
+
+
+def kerepel_kernels(torch, size: dict, peak: dict):
+    """Kerepel's kernels alone, replayed back to back on operands of their own, each followed by the like kernel of the
+    closest design at the same sizes (Deluvik's attention, router and experts, Fuvolix's latent attention): prompt
+    portions (2 x 1,024 tokens) and single tokens (8 requests at 1,023 cached tokens)."""
+    from mini_llm_b200.kernels import ops
+    lines = []
+    page, fma_peak = 64, FP32_FMA_TFLOPS_NOMINAL
+    dev = lambda values: torch.tensor(values, dtype=torch.int32, device="cuda")
+
+    def add(kernel, us, flops=None, bytes_moved=None, tensor_flops=None, **more):
+        line = {"kernel": kernel, "us": round(us, 2), **more}
+        if flops is not None:
+            line.update(tflops=round(flops / us / 1e6, 2), frac_fp32_fma_nominal=round(flops / us / 1e6 / fma_peak, 3))
+        if tensor_flops is not None:
+            line.update(tflops=round(tensor_flops / us / 1e6, 1), frac_bf16_measured=round(tensor_flops / us / 1e6 / peak["bf16_tflops"], 3))
+        if bytes_moved is not None:
+            line.update(gbs=round(bytes_moved / us / 1e3, 1), frac_hbm_measured=round(bytes_moved / us / 1e3 / peak["hbm_gbs"], 3))
+        lines.append(line)
+
+    att, lat, moe, width, taps = size["attention"], size["latent"], size["moe"], size["width"], size["taps"]
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    for name, lengths, new in (("prompts, 2 x 1024", [1024, 1024], [1024, 1024]), ("single tokens, 8 x 1024", [1024] * 8, [1] * 8)):
+        blocks = [-(-n // page) for n in lengths]
+        table = torch.stack([torch.arange(i * max(blocks), (i + 1) * max(blocks), dtype=torch.int32) for i in range(len(lengths))]).cuda()
+        n, single = sum(new), len(new) > 2
+        starts, offsets = [length - count for length, count in zip(lengths, new)], [sum(new[:i]) for i in range(len(new))]
+        positions = torch.cat([torch.arange(s, s + m) for s, m in zip(starts, new)]).int().cuda()
+        token_item = torch.cat([torch.full((m,), i) for i, m in enumerate(new)]).int().cuda()
+        items = (dev(list(range(len(new)))), dev(starts), dev(offsets), dev(new))
+        # ---- attention: a bias by distance and a gate per entry, beside a sink ----
+        heads, kv_heads, dim, vdim, window = att["heads"], att["kv_heads"], att["dim"], att["vdim"], size["window"]
+        scale, columns = dim ** -0.5, heads * dim + kv_heads * (dim + vdim)
+        k_pages = [torch.randn(sum(blocks) + 1, page, kv_heads, dim, device="cuda").bfloat16() for _ in range(4)]
+        v_pages = [torch.randn(sum(blocks) + 1, page, kv_heads, vdim, device="cuda").bfloat16() for _ in range(4)]
+        q = torch.randn(n, heads * dim, device="cuda").bfloat16()
+        out = torch.empty(n, heads * vdim, device="cuda", dtype=torch.bfloat16)
+        projected = [torch.randn(n, columns + heads * vdim, device="cuda") for _ in range(4)]
+        slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], device="cuda")
+        sink = torch.zeros(heads, device="cuda")
+        seen = sum(sum(min(p + 1, window) for p in range(s, s + m)) for s, m in zip(starts, new))
+        for like in ("", "(Deluvik) "):
+            extra = [dict(sink=sink) if like else dict(slopes=slopes, gate=one[:, columns:], gate_wide=True) for one in projected]
+            if single:
+                chunk = 128
+                chunks, row = -(-window // chunk), ops.split_attention_row(dim, vdim)
+                scratch = (torch.empty(n * heads * chunks * row, device="cuda"), torch.empty(n * heads * chunks * 2, device="cuda"),
+                           torch.zeros(n * heads, dtype=torch.int32, device="cuda"))
+                us = replayed_us(torch, lambda i: ops.split_attention(out, q, k_pages[i % 4], v_pages[i % 4], table, positions, token_item,
+                                                                      heads, kv_heads, dim, page, scale, window, chunk, chunks, *scratch,
+                                                                      cap=50.0, value_size=vdim, **extra[i % 4]))
+                add(f"{like}attention within {window}, split keys, {name}", us, bytes_moved=seen * kv_heads * (dim + vdim) * 2.0)
+            else:
+                us = replayed_us(torch, lambda i: ops.capped_attention(out, q, k_pages[i % 4], v_pages[i % 4], table, positions, token_item,
+                                                                       heads, kv_heads, dim, vdim, page, scale, 50.0, window, tiled=True,
+                                                                       **extra[i % 4]))
+                add(f"{like}attention within {window}, tiles, {name}", us, flops=2.0 * seen * heads * (dim + vdim))
+        weights = torch.randn(columns, taps, device="cuda")
+        states = [torch.zeros(len(new), taps - 1, columns, device="cuda") for _ in range(4)]
+        inv_freq = torch.tensor([10000.0 ** (-2.0 * i / dim) for i in range(dim // 2)], dtype=torch.float64, device="cuda")
+        moved = n * columns * 6.0 + 2.0 * len(new) * (taps - 1) * columns * 4
+        for label, norm, turned in (("taps, head norms and cache store", "head", 0),
+                                    ("(Deluvik) taps, norm, rotation and cache store", "whole", dim)):
+            gains = [torch.ones(dim if norm == "head" else h * dim, device="cuda") for h in (heads, kv_heads)]
+            us = replayed_us(torch, lambda i: ops.norm_rotary_store(projected[i % 4], heads * dim, (heads + kv_heads) * dim, heads, kv_heads, dim,
+                                                                    vdim, q, *gains, norm, 1e-5, turned, "half", inv_freq, positions, token_item,
+                                                                    table, page, k_pages[i % 4], v_pages[i % 4],
+                                                                    taps=(weights, states[i % 4], *items, single)))
+            add(f"{label}, {name}", us, bytes_moved=moved, columns=columns, taps=taps)
+        # ---- attention over the latent: a gate per head and scaled frequencies ----
+        heads, rank, rot, dim = lat["heads"], lat["kv_rank"], lat["rot_dim"], lat["dim"]
+        row = rank + rot
+        seen = sum(sum(p + 1 for p in range(s, s + m)) for s, m in zip(starts, new))
+        pages = [torch.randn(sum(blocks) + 1, page, 1, row, device="cuda").bfloat16() for _ in range(4)]
+        q_eff = torch.randn(n, heads * row, device="cuda")
+        q = torch.randn(n, heads * (dim + rot), device="cuda").bfloat16()
+        mixed = torch.empty(n, heads * rank, device="cuda", dtype=torch.bfloat16)
+        down = [torch.randn(n, row + heads, device="cuda") for _ in range(4)]
+        gain = torch.ones(rank, device="cuda")
+        inv_freq = torch.tensor([10000.0 ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float64, device="cuda")
+        for like in ("", "(Fuvolix) "):
+            gates = [None if like else one[:, row:] for one in down]
+            if single:
+                parts = max(1, min(32, 296 // n))
+                scratch = (torch.empty(n * heads * parts * rank, device="cuda"), torch.empty(n * heads * parts * 2, device="cuda"))
+                us = replayed_us(torch, lambda i: ops.latent_attention_tiled(mixed, q_eff, pages[i % 4], table, positions, token_item, heads, rank,
+                                                                             rot, page, 0.1, parts=parts, scratch=scratch, gate=gates[i % 4]))
+                add(f"{like}latent attention in parts, {name}", us, bytes_moved=seen * row * 2.0, heads=heads, row=row)
+            else:
+                tiles, _, _ = ops.attention_tiles(offsets, new, starts, split=False)
+                tiles_d = dev(tiles)
+                us = replayed_us(torch, lambda i: ops.latent_attention_tiled(mixed, q_eff, pages[i % 4], table, positions, token_item, heads, rank,
+                                                                             rot, page, 0.1, tiles=tiles_d, n_tiles=len(tiles), gate=gates[i % 4]))
+                add(f"{like}latent attention in tiles, {name}", us, flops=2.0 * seen * heads * (row + rank), heads=heads, row=row)
+            mine = [one[:, :row] if not like else one[:, :row].contiguous() for one in down]
+            us = replayed_us(torch, lambda i: ops.latent_prepare(pages[i % 4], q_eff, mine[i % 4], q, gain, inv_freq, positions, token_item, table,
+                                                                 page, rank, rot, rot, heads, dim, 1e-5, amplitude=1.0 if like else 1.2))
+            add(f"{like}latent norm, rotation and store, {name}", us, bytes_moved=n * (row * 6.0 + heads * rot * 6.0))
+        # ---- the router and the experts ----
+        experts, top, inner, shared = moe["experts"], moe["top"], moe["ff"], moe["shared"]
+        pairs, total = top + 1, moe["experts"] * moe["ff"] + moe["shared"]
+        x = torch.randn(n, width, device="cuda").bfloat16()
+        hidden = torch.zeros(n, width, device="cuda")
+        router = (torch.randn(experts, width, device="cuda") * 0.05).bfloat16()
+        opened = (torch.randn(1, width, device="cuda") * 0.05).bfloat16()
+        correction, bias = torch.randn(experts, device="cuda") * 0.02, torch.zeros(experts, device="cuda")
+        choice = torch.zeros(n * pairs, dtype=torch.int32, device="cuda")
+        in_weight, out_weight = torch.zeros(n * pairs, device="cuda"), torch.zeros(n * pairs, device="cuda")
+        up = [(torch.randn(2 * total, width, device="cuda") * 0.02).bfloat16() for _ in range(4)]
+        down = [(torch.randn(width, total, device="cuda") * 0.02).bfloat16() for _ in range(4)]
+        sizes = [inner] * experts + [shared]
+        first = [sum(sizes[:e]) for e in range(experts + 1)]
+        at = lambda base, places: torch.tensor([base + 2 * p for p in places], dtype=torch.int64, device="cuda")
+        tables = [(at(u.data_ptr(), [f * width for f in first]), at(u.data_ptr(), [(total + f) * width for f in first]), at(d.data_ptr(), first))
+                  for u, d in zip(up, down)]
+        for like in ("", "(Deluvik) "):
+            if like:
+                route = lambda i: ops.route(x, router, None, top, choice, in_weight, out_weight, bias=bias, rule="softmax_of_chosen",
+                                            shared_plain=True)
+                form = {}
+            else:
+                route = lambda i: ops.route(x, router, opened, top, choice, in_weight, out_weight, rule="sigmoid", correction=correction,
+                                            groups=moe["groups"], keep_groups=moe["keep"])
+                form = dict(form="clamped_glu", limit=7.0, shared_limit=7.0, alpha=1.702)
+            us = replayed_us(torch, route)
+            add(f"{like}router, {name}", us, bytes_moved=(n + experts) * width * 2.0, outputs=experts, top=top)
+            work = n * (top * inner + shared) * 3 * width
+            if single:
+                act = torch.empty(n * pairs, max(sizes), device="cuda", dtype=torch.bfloat16)
+                inner_of = dev(sizes)
+                us = replayed_us(torch, lambda i: ops.experts(hidden, act, x, choice, in_weight, out_weight, *tables[i % 4], inner_of, max(sizes),
+                                                              pairs, ld_down=total, n_experts=experts, **form))
+                used = sum(sizes[e] for e in set(choice.tolist()))
+                add(f"{like}experts, pair by pair, {name}", us, bytes_moved=used * 3 * width * 2.0)
+            else:
+                gu = torch.empty(n, 2 * total, device="cuda", dtype=torch.bfloat16)
+                act = torch.empty(n, total, device="cuda", dtype=torch.bfloat16)
+                combine = lambda i: ops.expert_combine(act, gu, choice, in_weight, out_weight, experts, inner, top, pairs, **form)
+
+                def launch(i):
+                    ops.gemm_bf16(gu, x, up[i % 4], None, "store", status)
+                    combine(i)
+                    ops.gemm_bf16(hidden, act, down[i % 4], None, "add", status)
+                us = replayed_us(torch, launch)
+                add(f"{like}experts, two products over all experts, {name}", us, tensor_flops=2.0 * work,
+                    executed_tflops=round(6.0 * n * width * total / us / 1e6, 1))
+                us = replayed_us(torch, combine)
+                add(f"{like}activation and weights between the products, {name}", us, bytes_moved=2.0 * n * (2 * (top * inner + shared) + total))
+        # ---- what the tokens' identities add ----
+        side, vocab = size["side"], GPT2_SMALL["vocab_size"]
+        ids = torch.randint(0, vocab, (n,), device="cuda", dtype=torch.int32)
+        embed = (torch.randn(vocab, width, device="cuda")).bfloat16()
+        pair_rows = (torch.randn(32750, width, device="cuda")).bfloat16()
+        last = torch.zeros(len(new), dtype=torch.int32, device="cuda")
+        us = replayed_us(torch, lambda i: ops.pair_embed(hidden, ids, positions, token_item, items[0], items[2], items[3], embed, pair_rows, last,
+                                                         32749, 10007, 31))
+        add(f"embedding with pair rows, {name}", us, bytes_moved=n * width * 8.0)
+        us = replayed_us(torch, lambda i: ops.embed(hidden, ids, positions, embed))
+        add(f"(Deluvik) embedding, {name}", us, bytes_moved=n * width * 6.0)
+        own = torch.randn(vocab, size["layers"] * side, device="cuda").bfloat16()
+        gate = [(torch.randn(side, width, device="cuda") * 0.02).bfloat16() for _ in range(4)]
+        proj = [(torch.randn(width, side, device="cuda") * 0.1).bfloat16() for _ in range(4)]
+        streams = [torch.randn(n, width, device="cuda") for _ in range(4)]
+        narrow, z = torch.empty(n, side, device="cuda", dtype=torch.bfloat16), torch.randn(n, side, device="cuda")
+        rounded, normed = (torch.empty(n, width, device="cuda", dtype=torch.bfloat16) for _ in range(2))
+        y, gain = torch.randn(n, width, device="cuda"), torch.ones(width, device="cuda")
+        if single:
+            us = replayed_us(torch, lambda i: ops.token_gate(narrow, streams[i % 4], gate[i % 4], own, ids, side))
+            add(f"token gate on the stream, {name}", us, bytes_moved=side * width * 2.0 + n * width * 4.0)
+            us = replayed_us(torch, lambda i: ops.skinny_linear(y, narrow, proj[i % 4]))
+            add(f"token side, back to the width, {name}", us, bytes_moved=side * width * 2.0 + n * width * 4.0)
+            us = replayed_us(torch, lambda i: ops.skinny_linear(z, rounded, gate[i % 4]))
+            add(f"(Deluvik) a product of the gate's size, {name}", us, bytes_moved=side * width * 2.0 + n * width * 2.0)
+        else:
+            us = replayed_us(torch, lambda i: ops.token_gate_rows(narrow, z, own, ids, side))
+            add(f"token gate behind its product, {name}", us, bytes_moved=n * side * 8.0)
+
+            def whole(i):
+                ops.add_normed_cast(streams[i % 4], act=rounded)
+                ops.gemm_bf16(z, rounded, gate[i % 4], None, "store", status)
+                ops.token_gate_rows(narrow, z, own, ids, side)
+                ops.gemm_bf16(y, narrow, proj[i % 4], None, "store", status)
+            us = replayed_us(torch, whole)
+            add(f"token side up to its result, {name}", us, bytes_moved=n * width * 12.0 + n * side * 14.0)
+        us = replayed_us(torch, lambda i: ops.add_normed_norm(streams[i % 4], y, gain, 1e-5, normed, gain, 1e-5))
+        add(f"normed sum with the next norm, {name}", us, bytes_moved=n * width * (4 + 4 + 4 + 2.0))
+        us = replayed_us(torch, lambda i: ops.add_normed_cast(streams[i % 4], y, gain, 1e-5, normed))
+        add(f"(Deluvik) normed sum with the rounded rows, {name}", us, bytes_moved=n * width * (4 + 4 + 4 + 2.0))
+    return lines
+
+
+def run_compare_kerepel(args):
+    """Kerepel beside Deluvik of equal width, depth, heads and feed-forward weights: the prompt step of 2,048 tokens (2 x
+    1,024) and the decode step of ``--batch`` requests at a context of 1,024, in bfloat16, through ``Engine.step``; then the
+    kernels alone, Kerepel's own and the closest designs' like ones.  One JSON line per measurement."""
+    import torch
+    from mini_llm_b200.config import config_from_dict
+    from mini_llm_b200.engine import Engine
+    from mini_llm_b200.weights import write_random_model
+    peak = peaks()
+    context, vocab = 1024, GPT2_SMALL["vocab_size"]
+    for name, size in KEREPEL_SIZES.items():
+        for design, raw in (("kerepel", kerepel_config(size, vocab)), ("deluvik", kerepel_like_config(size, vocab))):
+            with tempfile.TemporaryDirectory() as folder:
+                write_random_model(config_from_dict(raw), 0, folder, recipe="gpt2", store_dtype="bfloat16")
+                engine = Engine(folder, dtype="bfloat16", max_requests=16, cache_tokens=16 * context, max_tokens_per_step=2048,
+                                **({"page_size": args.page_size} if args.page_size else {}))
+                prefill_ms = prefill_run(engine, 2, 1024, vocab)
+                decode_ms, launches, _ = decode_run(engine, args.batch, args.steps, args.warmup, context, vocab)
+                print(json.dumps({"design": design, "size": name, "width": size["width"], "layers": size["layers"],
+                                  "prefill_2048_tokens_ms": round(prefill_ms, 3), "prefill_tokens_per_s": round(2048 / prefill_ms * 1e3),
+                                  "decode_batch": args.batch, "decode_ms_per_step": round(decode_ms, 3),
+                                  "decode_tokens_per_s": round(args.batch / decode_ms * 1e3), "launches_per_decode_step": launches,
+                                  "weight_bytes": engine.model.weight_bytes, "step_kinds": engine.step_kinds}), flush=True)
+                del engine
+                torch.cuda.empty_cache()
+        for line in kerepel_kernels(torch, size, peak):
+            print(json.dumps(dict(line, size=name)), flush=True)
+    return 0
+
+
 def run_compare(args):
     """Fuvolix beside GPT-2 of equal width, depth and inner size: the prompt step of 2,048 tokens
     (2 x 1,024) and the decode step of ``--batch`` requests at a context of 1,024, in bfloat16,
@@ -1754,6 +2026,8 @@ def main():
         return run_compare_deluvik(args)
     if args.compare == "nufavik":
         return run_compare_nufavik(args)
+    if args.compare == "kerepel":
+        return run_compare_kerepel(args)
     if args.compare:
         return run_compare(args)
     return run_ours(args)
