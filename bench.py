@@ -1742,7 +1742,7 @@ def kerepel_config(size: dict, vocab: int) -> dict:
 def kerepel_like_config(size: dict, vocab: int) -> dict:
     """Deluvik of equal width, depth, heads and feed-forward weights: attention over all keys where Kerepel has the latent."""
     att, lat, moe = size["attention"], size["latent"], size["moe"]
-    dense = {"kind": "dense", "ff": size["ff"] * 2 // 3}                     # (three matrices, not two)
+    dense = {"kind": "dense", "ff": (size["ff"] * 2 // 3 + 32) // 64 * 64}   # (three matrices, not two; a size the fast kernels take)
     routed = {"kind": "moe", "router": {"experts": moe["experts"], "top": moe["top"]}, "expert": {"ff": moe["ff"]},
               "shared": {"ff": moe["shared"]}}
     rot = {"base": 10000.0, "dims": att["dim"]}

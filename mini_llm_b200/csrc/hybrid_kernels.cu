@@ -531,6 +531,7 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
     float* weights = values + BLOCK_KEYS * vd;               // [64][pd]
     int* row_pos = reinterpret_cast<int*>(weights + BLOCK_ROWS * pd);     // [64]
     int* row_item = row_pos + BLOCK_ROWS;                    // [64]
+    float* row_slope = reinterpret_cast<float*>(row_item + BLOCK_ROWS);   // [64]
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     const int group = n_heads / n_kv_heads;
     const int chunks = (group + heads_per_block - 1) / heads_per_block;
@@ -550,6 +551,7 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
         const int token = live ? first_token + r / n_heads_here : 0;
         row_pos[r] = live ? positions[token] : -1;
         row_item[r] = live ? token_item[token] : -1;
+        row_slope[r] = live && slopes != nullptr ? slopes[first_head + r % n_heads_here] : 0.0f;
     }
     for (int u = tid; u < BLOCK_ROWS * (dim / VEC); u += blockDim.x) {
         const int r = u / (dim / VEC), d = (u % (dim / VEC)) * VEC;
@@ -561,11 +563,9 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
     __syncthreads();
     constexpr int RT = BLOCK_RT;
     int my_pos[RT], my_item[RT], my_first[RT];
-    float m[RT], l[RT], o[RT][4 * VG], slope[RT];
+    float m[RT], l[RT], o[RT][4 * VG];
 #pragma unroll
     for (int i = 0; i < RT; i++) {
-        const int r = ty * RT + i;
-        slope[i] = slopes != nullptr && r < n_rows ? slopes[first_head + r % n_heads_here] : 0.0f;
         my_pos[i] = row_pos[ty * RT + i], my_item[i] = row_item[ty * RT + i];
         my_first[i] = first_visible(my_pos[i], window, 0);
         m[i] = -INFINITY, l[i] = 0.0f;
@@ -668,12 +668,13 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
 #pragma unroll
             for (int i = 0; i < RT; i++) {
                 const bool row_here = my_item[i] == item;
+                const float slope = row_slope[ty * RT + i];
                 float score[4], top = -INFINITY;
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
                     const int pos = base + tx + 16 * j;
                     const bool seen = row_here && pos <= my_pos[i] && key_visible(pos, my_first[i], keep);
-                    score[j] = seen ? capped(acc[i][j] * scale, cap, inv_cap) - slope[i] * (float)(my_pos[i] - pos) : -INFINITY;
+                    score[j] = seen ? capped(acc[i][j] * scale, cap, inv_cap) - slope * (float)(my_pos[i] - pos) : -INFINITY;
                     top = fmaxf(top, score[j]);
                 }
 #pragma unroll
@@ -750,7 +751,7 @@ capped_attention_block_kernel(T* __restrict__ out, long ld_out, const T* __restr
 
 static size_t capped_block_shared(int dim, int vdim) {
     return sizeof(float) * ((size_t)2 * BLOCK_ROWS * (dim + 4) + (size_t)BLOCK_KEYS * (vdim + 4) + (size_t)BLOCK_ROWS * (BLOCK_KEYS + 4)) +
-           sizeof(int) * 2 * BLOCK_ROWS;
+           (2 * sizeof(int) + sizeof(float)) * BLOCK_ROWS;
 }
 
 // (keys and values in whole 16-byte vectors; values narrower than half their groups go to the tiles of few rows)
